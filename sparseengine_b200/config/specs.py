@@ -67,6 +67,8 @@ class RMSNormSpec:
     # the stored weight w is applied as (offset + w): 1.0 for weights kept around zero.  Such a norm keeps its
     # weight in 32-bit (the sum would lose the stored digits in a 16-bit type).
     offset: float = 0.0
+    # the row is split into this many equal parts, each divided by its own root mean square (over a 32-bit stream only)
+    groups: int = 1
 
 
 @dataclass(frozen=True)
@@ -88,7 +90,8 @@ class AttentionSpec:
     head_dim: int = 0
     scale: float = 1.0
     # None | "whole_projection" (one root mean square over all heads, a weight per column) | "per_head" (one per
-    # head, a weight of head_dim elements shared by the heads; needs prep="general")
+    # head, a weight of head_dim elements shared by the heads; needs prep="general") | "per_head_unit" (one per
+    # head, no weight; needs prep="general")
     qk_norm: Optional[str] = None
     qk_norm_eps: float = 1e-6
     window: Optional[int] = None      # keys p-window+1..p; None = all keys
@@ -108,6 +111,9 @@ class AttentionSpec:
     # with a window: the first keep_first positions stay visible to every later query (at their true positions),
     # beside the window's keys
     keep_first: int = 0
+    # a distance bias: one slope per query head; the scaled score of query position i and key position j loses
+    # slope * (i - j)
+    distance_slopes: Optional[tuple] = None
     # biases on the q, k, v rows of the packed projection (parameter ``qkv_bias``) and on the output projection
     # (``o_bias``); needs prep="general"
     bias: bool = False
@@ -209,12 +215,14 @@ class StreamMixSpec:
 class LatentAttentionSpec:
     """Softmax attention whose keys and values are up-projections of one cached latent per position.
 
-    Queries go through a latent of their own (``q_rank``, RMS-normed); a head's query and key have
+    Queries go through a latent of their own (``q_rank``, RMS-normed) or, with ``q_rank`` 0, come straight
+    from a projection of the input; a head's query and key have
     ``head_dim`` unrotated dims followed by ``rot_dim`` rotated ones.  The key/value projection gives
     ``kv_rank`` latent dims (RMS-normed) plus ``rot_dim`` dims that form the rotated key part of every
     head; unrotated keys and values are ``W_uk c`` and ``W_uv c``.  Only the latent and the rotated key
     part are cached.  ``window``: keys p-window+1..p (None: all).  ``sink``: a learned logit per head
-    that joins the softmax's denominator, unscaled, with no key or value."""
+    that joins the softmax's denominator, unscaled, with no key or value.  ``output_gate`` (needs ``q_rank``
+    0): the concatenated heads are multiplied by ``sigmoid(W_g x)`` before the output projection."""
     kind: str = "latent_attention"
     hidden_size: int = 0
     num_heads: int = 0
@@ -226,8 +234,9 @@ class LatentAttentionSpec:
     scale: float = 1.0
     window: Optional[int] = None
     sink: bool = False
-    position: Optional[Any] = None    # RotarySpec over (at most) rot_dim dims, split-half pairing
+    position: Optional[Any] = None    # RotarySpec over (at most) rot_dim dims, split-half or interleaved pairing
     norm_eps: float = 1e-6
+    output_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -244,6 +253,16 @@ class RetentionSpec:
     decays: tuple = ()                # one per head
     position: Optional[Any] = None    # RotarySpec, split-half pairing
     norm_eps: float = 1e-6
+
+
+@dataclass(frozen=True)
+class MinGRUSpec:
+    """A gated recurrence over ``width`` channels whose gates read the current token only (minGRU):
+    ``z = sigmoid(W_z x + b_z)``, ``u = W_x x + b_x``, candidate ``c = u + 1/2`` where ``u >= 0`` and ``sigmoid(u)``
+    elsewhere, ``S <- (1 - z) S + z c``; the result is ``W_o (S * silu(W_g x))``."""
+    kind: str = "mingru"
+    hidden_size: int = 0
+    width: int = 0
 
 
 @dataclass(frozen=True)
@@ -310,8 +329,8 @@ class LayerSpec:
     mixer_norm: Any
     feed_forward_norm: Any
     arrangement: str = "pre_norm"
-    # "pre_norm_stream": x <- x + mixer(norm(x)), x <- x + ff(norm(x)) over a 32-bit stream; the
-    # feed-forward (with its norm) may be None.
+    # "pre_norm_stream": x <- x + a * mixer(norm(x)), x <- x + a * ff(norm(x)) over a 32-bit stream, a =
+    # residual_scale; the feed-forward (with its norm) may be None.
     # "post_norm": x <- norm(residual_scale * x + sublayer(x)) for each sublayer; the feed-forward
     # (with its norm) may be None
     # "stream_mix": pre-norm over several 32-bit streams; extra["mixer_streams"] and extra["feed_forward_streams"]
@@ -338,6 +357,10 @@ class ScheduleEntry:
     layer: int
     cache: Optional[int] = None
     write_cache: bool = True
+    # Before this visit the embedding output is added to the stream (``add_embedding``), then row ``step_vector``
+    # of the model's ``step_source`` tensor [passes, width] (a looped stack that marks its passes).
+    add_embedding: bool = False
+    step_vector: Optional[int] = None
     # Before this visit the stream becomes W [x; x0], x0 being the embedding output and W the
     # model's ``reinject_source`` tensor [width, 2 width] (a looped stack takes the embedding in
     # again at the start of every pass).
@@ -367,5 +390,7 @@ class ModelSpec:
     # stream is 32-bit whatever the activation type; blocks carry (its copy in the activation type,
     # the stream), the embedding is scaled in 32-bit and the final norm reads the stream.
     residual_stream: str = "activation"
+    step_source: Optional[str] = None               # checkpoint name of the [passes, width] vectors of ScheduleEntry.step_vector
+    step_count: int = 0                             # its number of rows
     reinject_source: Optional[str] = None           # checkpoint name of the [width, 2 width] matrix of ScheduleEntry.reinject
     streams: int = 1                                # copies of the residual stream ("stream_mix" blocks); the last norm reads their sum

@@ -13,7 +13,7 @@
 //
 // Any page size; query/key head sizes 64 and 128, value head sizes 32, 64 and 128 (others use the
 // plain kernel); a window is honoured, with or without first keys that stay visible.  A page holds the keys [kv head][slot][D] and then the values
-// [kv head][slot][DV].  The softmax's options (a cap on the scores, a sink of score 0, an output gate)
+// [kv head][slot][DV].  The softmax's options (a cap on the scores, a sink, an output gate, a distance bias)
 // are those of mma_util.cuh's SoftmaxOptions; the sink joins once, where the last sum is taken (here
 // for one split, in the second kernel for several), and the gate where the output is rounded.
 // A block-table entry outside [0, num_pages) is not followed: the rows it stands for are
@@ -157,6 +157,16 @@ attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // w
                 mma_bf16(s[1], qa[kk], b2, b3);
             }
             if (opt.cap_in > 0.f) cap_scores<8>(&s[0][0], opt.cap_in, opt.cap_out);
+            if (opt.slopes != nullptr) {
+                // the distance bias of this lane's two rows (heads) per token
+                const float slope[2] = {g < rows_valid ? raw_slope(opt, head0 + g) : 0.f,
+                                        g + 8 < rows_valid ? raw_slope(opt, head0 + g + 8) : 0.f};
+#pragma unroll
+                for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        s[nt][e] = fmaf(slope[e >> 1], (float)(key_of(key0 + nt * 8 + 2 * t4 + (e & 1)) - pos), s[nt][e]);
+            }
             // mask keys beyond the range (rows share the token, hence the range)
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -339,7 +349,7 @@ extern "C" int se_attn_decode(const void* q, const void* cache, const int* table
                               float* part_o, float* part_ml, int tokens, int hq, int hkv, int head_dim, int v_head_dim,
                               int page_size, float scale, int window, int splits, int keys_per_split, int num_pages,
                               int* error, int settled, float softcap, int sink, const void* gate, int gate_pitch,
-                              const float* sink_logits, int keep_first, cudaStream_t stream) {
+                              const float* sink_logits, int keep_first, const float* slopes, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (!se_attn_decode_supported(head_dim, hq, hkv) || !se_attn_decode_value_dim_supported(v_head_dim) || splits < 1 ||
         keys_per_split <= 0 || keys_per_split % 64)
@@ -349,7 +359,7 @@ extern "C" int se_attn_decode(const void* q, const void* cache, const int* table
         return SE_ERR_ARGUMENT;
     const se::mma::SoftmaxOptions opt{softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f,
                                       sink || sink_logits != nullptr, (const __nv_bfloat16*)gate, gate_pitch, sink_logits,
-                                      window > 0 ? keep_first : 0};
+                                      window > 0 ? keep_first : 0, slopes, 1.f / scale};
 #define SE_DECODE_CASE(DQ, DVAL)                                                                                        \
     if (head_dim == DQ && v_head_dim == DVAL)                                                                           \
         return se::dec::launch<DQ, DVAL>(q, cache, table, table_stride, seq_rows, token_seq, positions, out, part_o,   \

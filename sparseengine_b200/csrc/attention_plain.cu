@@ -11,7 +11,8 @@
 // that has no value (one more term, exp(0), in the softmax's denominator); `gate` (with its row
 // pitch) multiplies the output element by element with sigmoid(gate[t][h * dv + i]); `sink_logits`
 // (one per query head) puts a learned logit in the place of the sink's 0, unscaled; `keep_first` n > 0
-// (with a window) keeps keys 0..n-1 visible beside the window's.  Reference: src/sparseengine/kernels/triton/context_flashattention_nopad.py:92-127,
+// (with a window) keeps keys 0..n-1 visible beside the window's; `slopes` (one per query head) takes
+// slope * (i - j) off the score of query position i and key position j.  Reference: src/sparseengine/kernels/triton/context_flashattention_nopad.py:92-127,
 // src/sparseengine/kernels/triton/gqa_flash_decoding_stage1.py:69-120.
 //
 // A block-table entry outside [0, num_pages) is not followed: the key is left out and a code
@@ -32,7 +33,8 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
                                              int d, int dv, int page_size, float scale, int window, int num_pages,
                                              int* __restrict__ error, float softcap, int sink,
                                              const T* __restrict__ gate, int gate_pitch,
-                                             const float* __restrict__ sink_logits, int keep_first) {
+                                             const float* __restrict__ sink_logits, int keep_first,
+                                             const float* __restrict__ slopes) {
     const int t = blockIdx.x, h = blockIdx.y;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int kvh = h / (hq / hkv);
@@ -52,6 +54,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
         acc[i] = 0.f;
     }
     float m = -INFINITY, l = 0.f;
+    const float slope = slopes != nullptr ? slopes[h] : 0.f;
     // the keys in the order they are visited: the kept first ones that lie before the window, then the window's
     const int kept = min(keep_first, lo), seen = kept + pos - lo + 1;
     for (int n = warp; n < seen; n += kAttnWarps) {
@@ -68,6 +71,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
         }
         s = warp_sum(s);
         if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+        s -= slope * (float)(pos - j);
         const float m_new = fmaxf(m, s);
         const float corr = expf(m - m_new);   // m = -inf on the first key: exp(-inf) = 0
         const float p = expf(s - m_new);
@@ -112,7 +116,7 @@ extern "C" int se_paged_attention_plain(const void* q, const void* cache, const 
                                         const int* seq_rows, const int* token_seq, const int* positions, void* out,
                                         int tokens, int hq, int hkv, int d, int dv, int page_size, float scale, int window,
                                         int num_pages, int* error, float softcap, int sink, const void* gate, int gate_pitch,
-                                        const float* sink_logits, int keep_first, int dtype, cudaStream_t stream) {
+                                        const float* sink_logits, int keep_first, const float* slopes, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (softcap < 0.f || (gate != nullptr && gate_pitch < hq * dv) || keep_first < 0) return SE_ERR_ARGUMENT;
     if (sink_logits != nullptr) sink = 1;
@@ -123,6 +127,6 @@ extern "C" int se_paged_attention_plain(const void* q, const void* cache, const 
         se::paged_attention_plain_kernel<T><<<grid, 32 * se::kAttnWarps, 0, stream>>>(
             (const T*)q, (const T*)cache, table, table_stride, seq_rows, token_seq, positions, (T*)out, hq, hkv, d, dv,
             page_size, scale, window, num_pages, error, softcap, sink, (const T*)gate, gate_pitch,
-            sink_logits, keep_first));
+            sink_logits, keep_first, slopes));
     SE_LAUNCH_CHECK();
 }

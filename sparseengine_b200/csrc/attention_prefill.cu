@@ -13,7 +13,7 @@
 //
 // Any page size; query/key head sizes 64 and 128, value head sizes 32, 64 and 128 (others use the
 // plain kernel): a page holds the keys [kv head][slot][D] and then the values [kv head][slot][DV].
-// The softmax's options (a cap on the scores, a sink of score 0, an output gate) are those of
+// The softmax's options (a cap on the scores, a sink, an output gate, a distance bias) are those of
 // mma_util.cuh's SoftmaxOptions.  A block-table entry outside [0, num_pages) is not followed: its
 // rows are zero-filled and a code goes to the error word.
 #include "common.cuh"
@@ -105,8 +105,12 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
     int lo[2];
+    float slope[2];                   // the distance bias of the row's head per token, in raw score units
 #pragma unroll
-    for (int h = 0; h < 2; ++h) lo[h] = window > 0 ? max(0, pos[h] - window + 1) : 0;
+    for (int h = 0; h < 2; ++h) {
+        lo[h] = window > 0 ? max(0, pos[h] - window + 1) : 0;
+        slope[h] = raw_slope(opt, head[h]);
+    }
 
     // Rows [64][DIM] of a tile: a thread copies chunk (tid % chunks) of rows tid / chunks + k * (kThreads / chunks).
     // The rows' addresses are looked up first (independent loads), so that no table load sits
@@ -182,6 +186,13 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
             }
         }
         if (opt.cap_in > 0.f) cap_scores<kTileKeys / 2>(&s[0][0], opt.cap_in, opt.cap_out);
+        if (opt.slopes != nullptr) {
+#pragma unroll
+            for (int n = 0; n < kTileKeys / 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    s[n][e] = fmaf(slope[e >> 1], (float)(key0 + n * 8 + 2 * t4 + (e & 1) - pos[e >> 1]), s[n][e]);
+        }
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int n = 0; n < kTileKeys / 8; ++n)
@@ -302,7 +313,8 @@ extern "C" int se_attn_prefill(const void* q, const void* cache, const int* tabl
                                const int* seq_rows, const int* cu_q, const int* kv_len, void* out, int entries,
                                int max_q_len, int hq, int hkv, int head_dim, int v_head_dim, int page_size, float scale,
                                int window, int num_pages, int* error, float softcap, int sink, const void* gate,
-                               int gate_pitch, const float* sink_logits, int keep_first, cudaStream_t stream) {
+                               int gate_pitch, const float* sink_logits, int keep_first, const float* slopes,
+                               cudaStream_t stream) {
     if (entries <= 0 || max_q_len <= 0) return 0;
     if (!(head_dim == 64 || head_dim == 128) || hkv <= 0 || hq % hkv || entries > 65535 || hkv > 65535)
         return SE_ERR_UNSUPPORTED;
@@ -310,7 +322,7 @@ extern "C" int se_attn_prefill(const void* q, const void* cache, const int* tabl
         return SE_ERR_ARGUMENT;
     const se::mma::SoftmaxOptions opt{softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f,
                                       sink || sink_logits != nullptr, (const __nv_bfloat16*)gate, gate_pitch, sink_logits,
-                                      window > 0 ? keep_first : 0};
+                                      window > 0 ? keep_first : 0, slopes, 1.f / scale};
 #define SE_PREFILL_CASE(DQ, DVAL)                                                                                      \
     if (head_dim == DQ && v_head_dim == DVAL)                                                                          \
         return se::pre::launch<DQ, DVAL>(q, cache, table, table_stride, seq_rows, cu_q, kv_len, out, entries, max_q_len, \

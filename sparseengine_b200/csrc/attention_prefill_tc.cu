@@ -31,8 +31,8 @@
 // stage is free again when both issuers have committed its P·V.  Every mbarrier wait is
 // bounded and reports through the error word.  The softmax's options (a cap on the scores, a sink
 // of score 0, an output gate; mma_util.cuh's SoftmaxOptions) cost the softmax warps two more
-// special-function operations per score for the cap, one term in the last sum for the sink, and one
-// load and exponential per output element for the gate.  Arithmetic as the reference's prefill kernel
+// special-function operations per score for the cap, an add and a multiply-add per score for a distance
+// bias, one term in the last sum for the sink, and one load and exponential per output element for the gate.  Arithmetic as the reference's prefill kernel
 // (src/sparseengine/kernels/triton/context_flashattention_nopad.py:92-127).
 #include "common.cuh"
 #include "mma_util.cuh"
@@ -331,6 +331,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         const int lo = window > 0 ? max(0, pos - window + 1) : 0;
         const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
         float m_ref = -INFINITY, l = 0.f;                  // reference maximum (log2 units), running sum
+        const float slope = se::mma::raw_slope(opt, kvh * group + rr % group);      // distance bias per token, raw units
         bool ok = true;
         for (int j = 0; j < num_tiles && ok; ++j) {
             const int b = j & 1;
@@ -354,6 +355,17 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             }
             const bool first = j < kept_tiles;
             const int key0 = first ? j * kKeys : k_begin + (j - kept_tiles) * kKeys;
+            if (opt.slopes != nullptr) {
+                // s + slope * (key - pos), two keys at a time (differences of positions are exact in 32-bit)
+                float2* s2 = reinterpret_cast<float2*>(sv);
+                const float d0 = (float)(key0 - pos);
+                float2 d = make_float2(d0, d0 + 1.f);
+#pragma unroll
+                for (int c = 0; c < 32; ++c) {
+                    s2[c] = se::mma::fma2(make_float2(slope, slope), d, s2[c]);
+                    d.x += 2.f; d.y += 2.f;
+                }
+            }
             // A tile every row of the warp sees in full needs no masking (rows ascend with the
             // lane: lane 0 has the smallest position, lane 31 the largest window start).  A tile of kept first keys
             // is seen by every row as far as it holds such keys; in a window's tile a key before the row's window is
@@ -492,7 +504,7 @@ extern "C" int se_attn_prefill_tc(const void* q, const void* cache, const int* t
                                   const int* seq_rows, const int* cu_q, const int* kv_len, void* out, int* error,
                                   int entries, int max_q_len, int hq, int hkv, int head_dim, int page_size, float scale,
                                   int window, int num_pages, float softcap, int sink, const void* gate, int gate_pitch,
-                                  const float* sink_logits, int keep_first, cudaStream_t stream) {
+                                  const float* sink_logits, int keep_first, const float* slopes, cudaStream_t stream) {
     using namespace se::fa;
     if (entries <= 0 || max_q_len <= 0) return 0;
     if (!se_attn_prefill_tc_supported(head_dim, hq, hkv) || entries > 65535 || hkv > 65535) return SE_ERR_UNSUPPORTED;
@@ -500,7 +512,7 @@ extern "C" int se_attn_prefill_tc(const void* q, const void* cache, const int* t
         return SE_ERR_ARGUMENT;
     const se::mma::SoftmaxOptions opt{softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f,
                                       sink || sink_logits != nullptr, (const __nv_bfloat16*)gate, gate_pitch, sink_logits,
-                                      window > 0 ? keep_first : 0};
+                                      window > 0 ? keep_first : 0, slopes, 1.f / scale};
     const size_t smem = (size_t)kTiles * kQBytes + kStages * kKVStageBytes + 1024;
     static bool configured = false;
     if (!configured) {

@@ -21,28 +21,45 @@ namespace se {
 #define SE_CODE_BAD_PAGE_LATENT_PREP 27
 #define SE_CODE_BAD_PAGE_LATENT_ATTN 28
 
+// Element i of a vector whose first `rotary_dim` dims are rotated by the position: pair k turns by pos * inv_freq[k]
+// and is (k, k + rotary_dim/2), or with `interleaved` (2k, 2k + 1); the rest passes.
+template <typename T>
+__device__ __forceinline__ float rotated_element(const T* x, int i, int pos, const float* __restrict__ inv_freq,
+                                                 int rotary_dim, int interleaved) {
+    if (i >= rotary_dim) return to_float(x[i]);
+    const int half = rotary_dim / 2;
+    const bool first = interleaved ? (i & 1) == 0 : i < half;
+    const int k = interleaved ? i >> 1 : (first ? i : i - half);
+    const int a = interleaved ? 2 * k : k, b = interleaved ? 2 * k + 1 : k + half;
+    float sn, cs;
+    sincosf((float)pos * inv_freq[k], &sn, &cs);
+    const float u = to_float(x[a]), w = to_float(x[b]);
+    return first ? u * cs - w * sn : w * cs + u * sn;
+}
+
 // One block per token.  proj row: [q latent (q_rank) | kv latent (rank) | shared key part (rot)].
-//   cq_out[t]           = rmsnorm(q latent) * q_w                      (activation type)
+//   cq_out[t]           = rmsnorm(q latent) * q_w                      (activation type; q_rank 0: queries have no latent)
 //   page row [0, rank)  = rmsnorm(kv latent) * kv_w
-//   page row [rank, ..) = the key part, its first `rotary_dim` dims rotated by the position
-//                         (dim i pairs with i + rotary_dim/2; angle = position * inv_freq[i])
+//   page row [rank, ..) = the key part, rotated by the position (rotated_element)
 template <typename T>
 __global__ void latent_prep_kernel(const T* proj, int proj_stride, const T* __restrict__ q_w, const T* __restrict__ kv_w,
                                    const float* __restrict__ inv_freq, const int* __restrict__ positions,
                                    const int* __restrict__ token_seq, const int* __restrict__ seq_rows,
                                    const int* __restrict__ table, int table_stride, T* cache, T* cq_out, int q_rank,
-                                   int rank, int rot, int rotary_dim, float eps, int page_size, int num_pages,
-                                   int write_cache, int* error) {
+                                   int rank, int rot, int rotary_dim, int interleaved, float eps, int page_size,
+                                   int num_pages, int write_cache, int* error) {
     __shared__ float scratch[33];
     const int t = blockIdx.x;
     const T* row = proj + (size_t)t * proj_stride;
     float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = to_float(row[i]); sq += v * v; }
     for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_float(row[q_rank + i]); sk += v * v; }
-    const float inv_q = 1.0f / sqrtf(block_sum(sq, scratch) / (float)q_rank + eps);
     const float inv_k = 1.0f / sqrtf(block_sum(sk, scratch) / (float)rank + eps);
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-        cq_out[(size_t)t * q_rank + i] = from_float<T>(to_float(row[i]) * inv_q * to_float(q_w[i]));
+    if (q_rank > 0) {
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = to_float(row[i]); sq += v * v; }
+        const float inv_q = 1.0f / sqrtf(block_sum(sq, scratch) / (float)q_rank + eps);
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
+            cq_out[(size_t)t * q_rank + i] = from_float<T>(to_float(row[i]) * inv_q * to_float(q_w[i]));
+    }
     if (!write_cache) return;
     const int pos = positions[t];
     const int page = table[(size_t)seq_rows[token_seq[t]] * table_stride + pos / page_size];
@@ -52,28 +69,18 @@ __global__ void latent_prep_kernel(const T* proj, int proj_stride, const T* __re
     for (int i = threadIdx.x; i < rank; i += blockDim.x)
         dst[i] = from_float<T>(to_float(row[q_rank + i]) * inv_k * to_float(kv_w[i]));
     const T* kr = row + q_rank + rank;
-    const int half = rotary_dim / 2;
-    for (int i = threadIdx.x; i < rot; i += blockDim.x) {
-        float v = to_float(kr[i]);
-        if (i < rotary_dim) {
-            const int j = i < half ? i : i - half;
-            float sn, cs;
-            sincosf((float)pos * inv_freq[j], &sn, &cs);
-            const float u = to_float(kr[j]), w = to_float(kr[j + half]);
-            v = i < half ? u * cs - w * sn : w * cs + u * sn;
-        }
-        dst[rank + i] = from_float<T>(v);
-    }
+    for (int i = threadIdx.x; i < rot; i += blockDim.x)
+        dst[rank + i] = from_float<T>(rotated_element(kr, i, pos, inv_freq, rotary_dim, interleaved));
 }
 
 constexpr int kLatWarps = 4;
 
 // One block per (token, head); a warp takes every fourth key, lane l the dims l, l + 32, ...
-// q_lat: float [heads, tokens, rank]; q: [tokens, heads * (d + rot)] in the activation type, of which
+// q_lat: float [heads, tokens, rank]; q: [tokens, heads * (d + rot)] in the activation type (rows q_pitch apart), of which
 // the last `rot` of each head are the rotated part (rotated here); out: [tokens, heads, rank].
 template <typename T, int NL>
-__global__ void latent_attention_plain_kernel(const float* __restrict__ q_lat, const T* __restrict__ q, int d,
-                                              const float* __restrict__ inv_freq, int rotary_dim,
+__global__ void latent_attention_plain_kernel(const float* __restrict__ q_lat, const T* __restrict__ q, int q_pitch, int d,
+                                              const float* __restrict__ inv_freq, int rotary_dim, int interleaved,
                                               const T* __restrict__ cache, const int* __restrict__ table,
                                               int table_stride, const int* __restrict__ seq_rows,
                                               const int* __restrict__ token_seq, const int* __restrict__ positions,
@@ -88,19 +95,9 @@ __global__ void latent_attention_plain_kernel(const float* __restrict__ q_lat, c
     float* qs = lat_smem;
     float* sacc = lat_smem + D;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) qs[i] = q_lat[((size_t)h * tokens + t) * rank + i] * scale;
-    const T* qr = q + ((size_t)t * heads + h) * (d + rot) + d;
-    const int half = rotary_dim / 2;
-    for (int i = threadIdx.x; i < rot; i += blockDim.x) {
-        float v = to_float(qr[i]);
-        if (i < rotary_dim) {
-            const int j = i < half ? i : i - half;
-            float sn, cs;
-            sincosf((float)pos * inv_freq[j], &sn, &cs);
-            const float u = to_float(qr[j]), w = to_float(qr[j + half]);
-            v = i < half ? u * cs - w * sn : w * cs + u * sn;
-        }
-        qs[rank + i] = v * scale;
-    }
+    const T* qr = q + (size_t)t * q_pitch + (size_t)h * (d + rot) + d;
+    for (int i = threadIdx.x; i < rot; i += blockDim.x)
+        qs[rank + i] = rotated_element(qr, i, pos, inv_freq, rotary_dim, interleaved) * scale;
     __syncthreads();
     float qreg[NL], acc[NL];
 #pragma unroll
@@ -164,32 +161,33 @@ extern "C" int se_latent_max_row() { return 32 * 32; }
 extern "C" int se_latent_prep(const void* proj, int proj_stride, const void* q_w, const void* kv_w, const float* inv_freq,
                               const int* positions, const int* token_seq, const int* seq_rows, const int* table,
                               int table_stride, void* cache, void* cq_out, int tokens, int q_rank, int rank, int rot,
-                              int rotary_dim, float eps, int page_size, int num_pages, int write_cache, int* error,
-                              int dtype, cudaStream_t stream) {
+                              int rotary_dim, int interleaved, float eps, int page_size, int num_pages, int write_cache,
+                              int* error, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (q_rank <= 0 || rank <= 0 || rot < 0 || rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || page_size <= 0)
+    if (q_rank < 0 || (q_rank > 0 && (q_w == nullptr || cq_out == nullptr)) || rank <= 0 || rot < 0 || rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || page_size <= 0)
         return SE_ERR_ARGUMENT;
     SE_DISPATCH_DTYPE(dtype, T,
         se::latent_prep_kernel<T><<<tokens, 128, 0, stream>>>((const T*)proj, proj_stride, (const T*)q_w, (const T*)kv_w,
             inv_freq, positions, token_seq, seq_rows, table, table_stride, (T*)cache, (T*)cq_out, q_rank, rank, rot,
-            rotary_dim, eps, page_size, num_pages, write_cache, error));
+            rotary_dim, interleaved, eps, page_size, num_pages, write_cache, error));
     SE_LAUNCH_CHECK();
 }
 
-extern "C" int se_latent_attention_plain(const float* q_lat, const void* q, int d, const float* inv_freq, int rotary_dim,
-                                         const void* cache, const int* table, int table_stride, const int* seq_rows,
+extern "C" int se_latent_attention_plain(const float* q_lat, const void* q, int q_pitch, int d, const float* inv_freq,
+                                         int rotary_dim, int interleaved, const void* cache, const int* table, int table_stride, const int* seq_rows,
                                          const int* token_seq, const int* positions, const float* sink, void* out,
                                          int tokens, int heads, int rank, int rot, int page_size, float scale, int window,
                                          int num_pages, int* error, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     const int D = rank + rot;
     if (rank <= 0 || rot < 0 || D > se_latent_max_row() || heads <= 0 || heads > 65535) return SE_ERR_UNSUPPORTED;
-    if (rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || d < 0 || page_size <= 0) return SE_ERR_ARGUMENT;
+    if (rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || d < 0 || page_size <= 0 || q_pitch < heads * (d + rot))
+        return SE_ERR_ARGUMENT;
     dim3 grid(tokens, heads);
     const size_t smem = (size_t)(D + se::kLatWarps * rank) * sizeof(float);
 #define SE_LAT_LAUNCH(NL)                                                                                             \
     se::latent_attention_plain_kernel<T, NL><<<grid, 32 * se::kLatWarps, smem, stream>>>(                             \
-        q_lat, (const T*)q, d, inv_freq, rotary_dim, (const T*)cache, table, table_stride, seq_rows, token_seq,        \
+        q_lat, (const T*)q, q_pitch, d, inv_freq, rotary_dim, interleaved, (const T*)cache, table, table_stride, seq_rows, token_seq,        \
         positions, sink, (T*)out, tokens, heads, rank, rot, page_size, scale, window, num_pages, error)
     SE_DISPATCH_DTYPE(dtype, T, {
         if (D <= 128) SE_LAT_LAUNCH(4);
@@ -227,8 +225,8 @@ constexpr int kThreads = 32 * kWarps;
 using namespace se::mma;
 
 // qfull[t, h, :] = [q_lat[h, t, :] | rotated part of q[t, h]] in bfloat16: the query rows as the tiled kernel reads them
-__global__ void latent_q_pack_kernel(const float* __restrict__ q_lat, const __nv_bfloat16* __restrict__ q, int d,
-                                     const float* __restrict__ inv_freq, int rotary_dim,
+__global__ void latent_q_pack_kernel(const float* __restrict__ q_lat, const __nv_bfloat16* __restrict__ q, int q_pitch,
+                                     int d, const float* __restrict__ inv_freq, int rotary_dim, int interleaved,
                                      const int* __restrict__ positions, __nv_bfloat16* __restrict__ qfull, int tokens,
                                      int heads, int rank, int rot) {
     const int t = blockIdx.x, h = blockIdx.y;
@@ -236,20 +234,10 @@ __global__ void latent_q_pack_kernel(const float* __restrict__ q_lat, const __nv
     __nv_bfloat16* dst = qfull + ((size_t)t * heads + h) * D;
     for (int i = threadIdx.x; i < rank; i += blockDim.x)
         dst[i] = __float2bfloat16_rn(q_lat[((size_t)h * tokens + t) * rank + i]);
-    const __nv_bfloat16* qr = q + ((size_t)t * heads + h) * (d + rot) + d;
-    const int half = rotary_dim / 2;
+    const __nv_bfloat16* qr = q + (size_t)t * q_pitch + (size_t)h * (d + rot) + d;
     const int pos = positions[t];
-    for (int i = threadIdx.x; i < rot; i += blockDim.x) {
-        float v = __bfloat162float(qr[i]);
-        if (i < rotary_dim) {
-            const int j = i < half ? i : i - half;
-            float sn, cs;
-            sincosf((float)pos * inv_freq[j], &sn, &cs);
-            const float u = __bfloat162float(qr[j]), w = __bfloat162float(qr[j + half]);
-            v = i < half ? u * cs - w * sn : w * cs + u * sn;
-        }
-        dst[rank + i] = __float2bfloat16_rn(v);
-    }
+    for (int i = threadIdx.x; i < rot; i += blockDim.x)
+        dst[rank + i] = __float2bfloat16_rn(rotated_element(qr, i, pos, inv_freq, rotary_dim, interleaved));
 }
 
 // D16T, RT: the row's 16-dim groups rounded up to a multiple of four (the tile's chunks between the row's end and that
@@ -542,13 +530,14 @@ extern "C" int se_latent_attention_tiled_supported(int rank, int rot) {
     return rank > 0 && rot >= 0 && rank % 16 == 0 && rot % 16 == 0 && rank + rot <= 256;
 }
 
-extern "C" int se_latent_q_pack(const float* q_lat, const void* q, int d, const float* inv_freq, int rotary_dim,
-                                const int* positions, void* qfull, int tokens, int heads, int rank, int rot,
+extern "C" int se_latent_q_pack(const float* q_lat, const void* q, int q_pitch, int d, const float* inv_freq,
+                                int rotary_dim, int interleaved, const int* positions, void* qfull, int tokens, int heads, int rank, int rot,
                                 cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (heads <= 0 || heads > 65535 || rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1)) return SE_ERR_ARGUMENT;
+    if (heads <= 0 || heads > 65535 || rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || q_pitch < heads * (d + rot))
+        return SE_ERR_ARGUMENT;
     se::lat::latent_q_pack_kernel<<<dim3(tokens, heads), 64, 0, stream>>>(
-        q_lat, (const __nv_bfloat16*)q, d, inv_freq, rotary_dim, positions, (__nv_bfloat16*)qfull, tokens, heads, rank, rot);
+        q_lat, (const __nv_bfloat16*)q, q_pitch, d, inv_freq, rotary_dim, interleaved, positions, (__nv_bfloat16*)qfull, tokens, heads, rank, rot);
     SE_LAUNCH_CHECK();
 }
 

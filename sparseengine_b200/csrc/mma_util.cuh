@@ -52,6 +52,9 @@ template <int D> __device__ __forceinline__ uint32_t tile_off(int r, int c) {
 //                     (rows gate_pitch elements apart); nullptr: no gate.
 //   sink_logits     : with `sink`, a learned logit per query head in the place of the sink's 0 (unscaled); nullptr: 0.
 //   keep_first      : with a window, keys 0 .. keep_first-1 stay visible beside the window's.
+//   slopes          : a distance bias: the scaled score of query position i and key position j becomes
+//                     s - slopes[query head] * (i - j); nullptr: none.  In raw units the bias per token is
+//                     slope * inv_scale.
 struct SoftmaxOptions {
     float cap_in, cap_out;
     int sink;
@@ -59,7 +62,13 @@ struct SoftmaxOptions {
     int gate_pitch;
     const float* sink_logits;
     int keep_first;
+    const float* slopes;
+    float inv_scale;
 };
+// what a head's raw scores lose per token of distance
+__device__ __forceinline__ float raw_slope(const SoftmaxOptions& opt, int head) {
+    return opt.slopes != nullptr ? opt.slopes[head] * opt.inv_scale : 0.f;
+}
 // the sink's logit of a head, times log2(e)
 __device__ __forceinline__ float sink_log2(const SoftmaxOptions& opt, int head) {
     return opt.sink_logits != nullptr ? opt.sink_logits[head] * 1.4426950408889634f : 0.f;

@@ -41,6 +41,7 @@ def library():
 # what the compiled library reports through `limit`).
 LIMITS = {
     "rmsnorm_max_width": 51200,             # a row is kept in shared memory in 32-bit
+    "rmsnorm_stream_max_groups": 4096,      # a partial sum per group in shared memory beside the row
     "router_max_experts": 12800,            # four floats per expert in shared memory during selection
     "router_max_unaligned_width": 6400,     # widths that are no multiple of 4 keep 8 token rows in shared memory
     "moe_max_experts": 6079,                # the routing build's scans keep two ints per expert in shared memory
@@ -50,8 +51,8 @@ LIMITS = {
     "latent_max_row": 1024,                 # latent plus shared key part of one position (32 registers x 32 lanes)
     "retention_max_head_dim": 256,          # rows of a retention state (32 registers x 8 warps)
     "stream_mix_max_streams": 16,           # a column's stream values live in registers
-    "memory_max_head_dim": 256,
-    "delta_chunk_max_head_dim": 256,        # a chunk's transposed q and k tiles in shared memory             # rows of a matrix memory's state (32 registers x 8 warps)
+    "memory_max_head_dim": 256,             # rows of a matrix memory's state (32 registers x 8 warps)
+    "delta_chunk_max_head_dim": 256,        # a chunk's transposed q and k tiles in shared memory
     "grid_dim_yz": 65535,                   # heads, KV heads and a step's entries map to grid dimensions y and z
 }
 
@@ -84,6 +85,15 @@ def _ptr(t: Optional[torch.Tensor], dtype=None, name: str = "tensor") -> Optiona
         raise ValueError(f"{name} must be a CUDA tensor (there is no CPU path)")
     if not t.is_contiguous():
         raise ValueError(f"{name} must be contiguous")
+    if dtype is not None and t.dtype != dtype:
+        raise TypeError(f"{name} must be {dtype}, got {t.dtype}")
+    return t.data_ptr()
+
+
+def _rows_ptr(t: torch.Tensor, name: str, dtype=None) -> int:
+    """The pointer of a CUDA matrix with contiguous rows (which may lie ``t.stride(0)`` elements apart)."""
+    if not t.is_cuda or t.dim() != 2 or t.stride(1) != 1:
+        raise ValueError(f"{name} must be a CUDA matrix with contiguous rows")
     if dtype is not None and t.dtype != dtype:
         raise TypeError(f"{name} must be {dtype}, got {t.dtype}")
     return t.data_ptr()
@@ -200,34 +210,44 @@ def _sink_logits(sink, num_heads: int):
     return _ptr(sink, torch.float32, "sink")
 
 
+def _slopes_ptr(slopes, num_heads: int):
+    if slopes is not None and slopes.shape != (num_heads,):
+        raise ValueError(f"a distance bias has one slope per query head ({num_heads}), got {tuple(slopes.shape)}")
+    return _ptr(slopes, torch.float32, "slopes")
+
+
 def paged_attention_plain(q, cache, table, seq_rows, token_seq, positions, out, *, num_heads, num_kv_heads,
                           head_dim, page_size, scale, window=None, num_pages=None, v_head_dim=None, softcap=None,
-                          sink=False, gate=None, keep_first: int = 0):
+                          sink=False, gate=None, keep_first: int = 0, slopes=None):
     """``v_head_dim``: the values' head size where it differs from the queries' and keys'.
     ``softcap`` c: scaled scores become c tanh(s / c).  ``sink``: True: a key of score 0 without a value
     joins the softmax's denominator; a 32-bit tensor [num_heads]: its logit is the head's entry (unscaled).
     ``gate``: a matrix (rows may be a view with a pitch) whose sigmoid multiplies the output,
-    [tokens, num_heads * v_head_dim].  ``keep_first`` n (with a window): keys 0..n-1 stay visible."""
+    [tokens, num_heads * v_head_dim].  ``keep_first`` n (with a window): keys 0..n-1 stay visible.
+    ``slopes`` (32-bit, [num_heads]): the score of query position i and key position j loses
+    ``slopes[head] * (i - j)``."""
     tokens = q.shape[0]
     dt = q.dtype
     if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1 or gate.dtype != dt):
         raise ValueError("gate must be a matrix of q's dtype with contiguous rows")
     sink_logits = _sink_logits(sink, num_heads)
-    _check(_fn("se_paged_attention_plain", "pppipppp" "iiiiii" "f" "iip" "fipi" "pi" "ip")(
+    _check(_fn("se_paged_attention_plain", "pppipppp" "iiiiii" "f" "iip" "fipi" "pip" "ip")(
         _ptr(q, None, "q"), _ptr(cache, dt, "cache"), _ptr(table, torch.int32, "table"), table.shape[1],
         _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(token_seq, torch.int32, "token_seq"),
         _ptr(positions, torch.int32, "positions"), _ptr(out, dt, "out"), tokens, num_heads, num_kv_heads,
         head_dim, int(v_head_dim or head_dim), page_size, float(scale), int(window or 0),
         cache.shape[0] if num_pages is None else int(num_pages), _ptr(error_word(q.device)),
         float(softcap or 0.0), _has_sink(sink), gate.data_ptr() if gate is not None else None,
-        gate.stride(0) if gate is not None else 0, sink_logits, int(keep_first or 0), dtype_code(dt), _stream()),
+        gate.stride(0) if gate is not None else 0, sink_logits, int(keep_first or 0), _slopes_ptr(slopes, num_heads),
+        dtype_code(dt), _stream()),
         "paged_attention_plain")
     return out
 
 
 def qk_prep_general(proj, q_w, k_w, positions, token_seq, seq_rows, table, cache, q_out, *, num_heads, num_kv_heads,
                     head_dim, v_head_dim, eps, page_size, has_kv=True, temperature=None, num_pages=None,
-                    inv_freq=None, rotary_dim: int = 0, v_first=None, v_mix=None, bias=None, per_head: bool = False):
+                    inv_freq=None, rotary_dim: int = 0, v_first=None, v_mix=None, bias=None, per_head: bool = False,
+                    per_head_unit: bool = False):
     """Query/key preparation in 32-bit, rounded once: whole-projection RMS norms (optional), a rotation
     of the first ``rotary_dim`` dims of every head (split halves, angles ``position * inv_freq``), a query
     temperature ``(coef, every)`` (q times 1 + coef ln(floor((p+1)/every) + 1)), keys and values of
@@ -235,8 +255,11 @@ def qk_prep_general(proj, q_w, k_w, positions, token_seq, seq_rows, table, cache
     ``v_first`` (a matrix with contiguous rows, [tokens, kv heads * v_head_dim]) and ``v_mix`` (one 32-bit
     number on the device): the values written are ``(1 - v_mix) v + v_mix v_first``.
     ``bias`` (32-bit, one per column of the projection row): added before anything else.  ``per_head``: the
-    norms are per head, with weights of ``head_dim`` elements shared by the heads."""
+    norms are per head, with weights of ``head_dim`` elements shared by the heads; ``per_head_unit``: per head
+    without weights."""
     tokens = proj.shape[0]
+    if per_head_unit and (per_head or q_w is not None or k_w is not None):
+        raise ValueError("qk_prep_general: per_head_unit is a norm without weights")
     if bias is not None and bias.numel() != num_heads * head_dim + (num_kv_heads * (head_dim + int(v_head_dim)) if has_kv else 0):
         raise ValueError("qk_prep_general: the bias has one entry per column of the projection row")
     dt = proj.dtype
@@ -254,7 +277,7 @@ def qk_prep_general(proj, q_w, k_w, positions, token_seq, seq_rows, table, cache
         _ptr(cache, dt, "cache") if has_kv else None, _ptr(q_out, dt, "q_out"), tokens, num_heads, num_kv_heads, head_dim,
         int(v_head_dim), float(eps), coef, every, page_size, int(bool(has_kv)),
         (cache.shape[0] if num_pages is None else int(num_pages)) if has_kv else 0, _ptr(error_word(proj.device)),
-        _ptr(bias, torch.float32, "bias"), int(bool(per_head)), dtype_code(dt), _stream()), "qk_prep_general")
+        _ptr(bias, torch.float32, "bias"), 2 if per_head_unit else int(bool(per_head)), dtype_code(dt), _stream()), "qk_prep_general")
     return q_out
 
 
@@ -303,17 +326,37 @@ def softcap_(x, cap: float):
     return x
 
 
-def add_rmsnorm_stream(x, y, w, eps: float, out32=None, out_act=None):
-    """A pre-norm model's 32-bit stream: ``v = x + y`` (``y`` optional, activation type) goes to
-    ``out32`` (which may be ``x``); ``out_act`` receives ``v / sqrt(mean(v^2) + eps) * w``, or, without
-    a weight, ``v`` rounded to the activation type."""
+def add_rmsnorm_stream(x, y, w, eps: float, out32=None, out_act=None, alpha: float = 1.0, groups: int = 1, inject=None):
+    """A pre-norm model's 32-bit stream: ``v = x + alpha * y`` (``y`` optional, activation type) goes to
+    ``out32`` (which may be ``x``); ``out_act`` receives ``v / sqrt(mean(v^2) + eps) * w`` (the mean over
+    each of ``groups`` equal parts of the row), or, without a weight, ``v`` rounded to the activation type.
+    ``inject``: ``(table, ids, scale, step)``: ``v`` also takes in ``table[ids[row]] * scale`` (``table`` None:
+    nothing) and the 32-bit vector ``step`` (or None)."""
     rows, hidden = x.shape
     dt = out_act.dtype if out_act is not None else (y.dtype if y is not None else torch.float32)
     if w is not None and w.shape != (hidden,):
         raise ValueError(f"norm weight shape {tuple(w.shape)} does not match width {hidden}")
-    _check(_fn("se_add_rmsnorm_stream", "ppppp" "ii" "f" "ip")(
-        _ptr(x, torch.float32, "x"), _ptr(y, dt, "y"), _ptr(w, dt, "w"), _ptr(out32, torch.float32, "out32"),
-        _ptr(out_act, dt, "out_act"), rows, hidden, float(eps), dtype_code(dt), _stream()), "add_rmsnorm_stream")
+    table, ids, scale, step = inject if inject is not None else (None, None, 0.0, None)
+    if table is not None and (table.shape[1] != hidden or ids.shape[0] != rows):
+        raise ValueError("inject: the table's rows must have the stream's width, and every row an id")
+    if step is not None and step.numel() != hidden:
+        raise ValueError("inject: the step vector must have the stream's width")
+    _check(_fn("se_add_rmsnorm_stream", "pp" "f" "ppp" "ii" "fi" "ppifp" "ip")(
+        _ptr(x, torch.float32, "x"), _ptr(y, dt, "y"), float(alpha), _ptr(w, dt, "w"), _ptr(out32, torch.float32, "out32"),
+        _ptr(out_act, dt, "out_act"), rows, hidden, float(eps), int(groups), _ptr(table, dt, "inject table"),
+        _ptr(ids, torch.int32, "inject ids"), table.shape[0] if table is not None else 0, float(scale),
+        _ptr(step, torch.float32, "inject step"), dtype_code(dt), _stream()), "add_rmsnorm_stream")
+
+
+def sigmoid_gate_(x, gate):
+    """x <- x * sigmoid(gate) in place (32-bit arithmetic, rounded once); ``gate`` may be a view of columns of a
+    projection (rows ``gate.stride(0)`` apart)."""
+    rows, width = x.shape
+    if gate.shape != x.shape or gate.dtype != x.dtype or gate.stride(1) != 1:
+        raise ValueError("sigmoid_gate: the gate must have x's shape and type and contiguous rows")
+    _check(_fn("se_sigmoid_gate", "pp" "iii" "ip")(_ptr(x, None, "x"), gate.data_ptr(), gate.stride(0), rows, width,
+                                                  dtype_code(x.dtype), _stream()), "sigmoid_gate")
+    return x
 
 
 def rmsnorm_add_stream(stream, y, w, eps: float, out_act=None):
@@ -331,34 +374,43 @@ def rmsnorm_add_stream(stream, y, w, eps: float, out_act=None):
 
 # ---- attention over a cached latent (csrc/latent_attention.cu) -----------------------------------
 
+def _interleaved(pairing: str) -> int:
+    if pairing not in ("split_half", "interleaved"):
+        raise ValueError(f"rotary pairing {pairing!r} is not supported by this kernel ('split_half' or 'interleaved')")
+    return int(pairing == "interleaved")
+
+
 def latent_prep(proj, q_w, kv_w, inv_freq, positions, token_seq, seq_rows, table, cache, cq_out, *, q_rank, rank, rot,
-                rotary_dim, eps, page_size, write_cache=True, num_pages=None):
+                rotary_dim, eps, page_size, write_cache=True, num_pages=None, pairing: str = "split_half"):
     """From a step's rows ``[q latent | kv latent | shared key part]``: the normalised query latent
-    (``cq_out``), and into each token's page slot the normalised kv latent and the rotated key part."""
+    (``cq_out``; ``q_rank`` 0: there is none), and into each token's page slot the normalised kv latent and
+    the rotated key part."""
     tokens = proj.shape[0]
     dt = proj.dtype
     if proj.dim() != 2 or proj.stride(1) != 1 or proj.shape[1] != q_rank + rank + rot:
         raise ValueError("proj must be [tokens, q_rank + rank + rot] with contiguous rows")
-    _check(_fn("se_latent_prep", "pippp" "ppp" "pi" "pp" "iiiii" "f" "iii" "p" "ip")(
+    _check(_fn("se_latent_prep", "pippp" "ppp" "pi" "pp" "iiiiii" "f" "iii" "p" "ip")(
         proj.data_ptr(), proj.stride(0), _ptr(q_w, dt, "q_norm"), _ptr(kv_w, dt, "kv_norm"),
         _ptr(inv_freq, torch.float32, "inv_freq"), _ptr(positions, torch.int32, "positions"),
         _ptr(token_seq, torch.int32, "token_seq"), _ptr(seq_rows, torch.int32, "seq_rows"),
         _ptr(table, torch.int32, "table"), table.shape[1], _ptr(cache, dt, "cache"), _ptr(cq_out, dt, "cq_out"),
-        tokens, q_rank, rank, rot, rotary_dim, float(eps), page_size,
+        tokens, q_rank, rank, rot, rotary_dim, _interleaved(pairing), float(eps), page_size,
         cache.shape[0] if num_pages is None else int(num_pages), int(bool(write_cache)), _ptr(error_word(proj.device)),
         dtype_code(dt), _stream()), "latent_prep")
     return cq_out
 
 
 def latent_attention_plain(q_lat, q, inv_freq, cache, table, seq_rows, token_seq, positions, sink, out, *, heads,
-                           head_dim, rank, rot, rotary_dim, page_size, scale, window=None, num_pages=None):
+                           head_dim, rank, rot, rotary_dim, page_size, scale, window=None, num_pages=None,
+                           pairing: str = "split_half"):
     """``q_lat`` float32 [heads, tokens, rank] (queries taken into the latent's space), ``q`` [tokens,
-    heads * (head_dim + rot)] whose rotated parts are rotated here; ``out`` [tokens, heads, rank]."""
+    heads * (head_dim + rot)] (rows may be a view with a pitch) whose rotated parts are rotated here; ``out``
+    [tokens, heads, rank]."""
     tokens = q.shape[0]
     dt = q.dtype
-    _check(_fn("se_latent_attention_plain", "ppipi" "ppi" "pppp" "p" "iiii" "i" "f" "ii" "p" "ip")(
-        _ptr(q_lat, torch.float32, "q_lat"), _ptr(q, None, "q"), head_dim, _ptr(inv_freq, torch.float32, "inv_freq"),
-        rotary_dim, _ptr(cache, dt, "cache"), _ptr(table, torch.int32, "table"), table.shape[1],
+    _check(_fn("se_latent_attention_plain", "ppiipii" "ppi" "pppp" "p" "iiii" "i" "f" "ii" "p" "ip")(
+        _ptr(q_lat, torch.float32, "q_lat"), _rows_ptr(q, "q"), q.stride(0), head_dim, _ptr(inv_freq, torch.float32, "inv_freq"),
+        rotary_dim, _interleaved(pairing), _ptr(cache, dt, "cache"), _ptr(table, torch.int32, "table"), table.shape[1],
         _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(token_seq, torch.int32, "token_seq"),
         _ptr(positions, torch.int32, "positions"), _ptr(sink, torch.float32, "sink"), _ptr(out, dt, "out"),
         tokens, heads, rank, rot, page_size, float(scale), int(window or 0),
@@ -373,12 +425,14 @@ def latent_attention_tiled_supported(rank: int, rot: int) -> bool:
     return rank > 0 and rot >= 0 and rank % 16 == 0 and rot % 16 == 0 and rank + rot <= 256
 
 
-def latent_q_pack(q_lat, q, inv_freq, positions, qfull, *, heads, head_dim, rank, rot, rotary_dim):
-    """``qfull[t, h] = [q_lat[h, t] | rotated part of q[t, h]]`` in bfloat16: the query rows of the tiled kernel."""
+def latent_q_pack(q_lat, q, inv_freq, positions, qfull, *, heads, head_dim, rank, rot, rotary_dim,
+                  pairing: str = "split_half"):
+    """``qfull[t, h] = [q_lat[h, t] | rotated part of q[t, h]]`` in bfloat16: the query rows of the tiled kernel.
+    ``q``'s rows may be a view with a pitch."""
     tokens = q.shape[0]
-    _check(_fn("se_latent_q_pack", "ppipi" "pp" "iiii" "p")(
-        _ptr(q_lat, torch.float32, "q_lat"), _ptr(q, torch.bfloat16, "q"), head_dim, _ptr(inv_freq, torch.float32, "inv_freq"),
-        rotary_dim, _ptr(positions, torch.int32, "positions"), _ptr(qfull, torch.bfloat16, "qfull"), tokens, heads, rank,
+    _check(_fn("se_latent_q_pack", "ppiipii" "pp" "iiii" "p")(
+        _ptr(q_lat, torch.float32, "q_lat"), _rows_ptr(q, "q", torch.bfloat16), q.stride(0), head_dim,
+        _ptr(inv_freq, torch.float32, "inv_freq"), rotary_dim, _interleaved(pairing), _ptr(positions, torch.int32, "positions"), _ptr(qfull, torch.bfloat16, "qfull"), tokens, heads, rank,
         rot, _stream()), "latent_q_pack")
     return qfull
 
@@ -640,6 +694,35 @@ def memory_out(o, gates, proj, g_off: int, w, out, *, heads, v_head_dim, eps: fl
         _ptr(o, torch.float32, "o"), _ptr(gates, torch.float32, "gates"), proj.data_ptr(), proj.stride(0), int(g_off),
         _ptr(w, torch.float32, "w"), out.data_ptr(), out.stride(0), tokens, heads, v_head_dim, float(eps),
         float(den_eps), float(out_scale), dtype_code(out.dtype), _stream()), "memory_out")
+    return out
+
+
+# ---- minGRU (csrc/min_gru.cu) ----------------------------------------------------------------
+
+def min_gru_scan(proj, bias, state, step, out):
+    """``proj`` [tokens, 3 * width] = ``[z' | u' | g]``; ``z = sigmoid(z' + b_z)``, ``u = u' + b_u``, the candidate is
+    ``u + 1/2`` (``u >= 0``) or ``sigmoid(u)``; ``S <- (1 - z) S + z * candidate``; ``out = S * silu(g)``.  ``bias`` [2 * width]
+    and ``state[row]`` [width] are 32-bit.  Token by token."""
+    width = out.shape[1]
+    _check(_fn("se_min_gru_scan", "pip" "pl" "ppp" "iii" "p")(
+        _rows_ptr(proj, "proj"), proj.stride(0), _ptr(bias, torch.float32, "bias"), _ptr(state, torch.float32, "state"),
+        state.stride(0), _ptr(step.cu_q), _ptr(step.seq_rows), _ptr(out, proj.dtype, "out"), step.num_seqs, width,
+        dtype_code(proj.dtype), _stream()), "min_gru_scan")
+    return out
+
+
+def min_gru_chunk(proj, bias, state, step, out, ctas=None):
+    """:func:`min_gru_scan` with a request's tokens dealt out to the warps of a cluster of ``ctas`` CTAs (128 tokens each
+    at a time; default: as many as the longest entry fills, at most 8): for steps with prompt portions."""
+    width = out.shape[1]
+    if ctas is None:
+        ctas = 1
+        while ctas < 8 and ctas * 128 < step.max_q_len:
+            ctas *= 2
+    _check(_fn("se_min_gru_chunk", "pip" "pl" "ppp" "iiii" "p")(
+        _rows_ptr(proj, "proj"), proj.stride(0), _ptr(bias, torch.float32, "bias"), _ptr(state, torch.float32, "state"),
+        state.stride(0), _ptr(step.cu_q), _ptr(step.seq_rows), _ptr(out, proj.dtype, "out"), step.num_seqs, width, int(ctas),
+        dtype_code(proj.dtype), _stream()), "min_gru_chunk")
     return out
 
 
@@ -1004,19 +1087,15 @@ def attn_decode_plan(tokens: int, num_heads: int, num_kv_heads: int, max_keys: i
     return splits, per_tiles * 64
 
 
-def _softmax_options(q, gate, num_heads, v_head_dim, softcap, sink, keep_first=None):
-    """The tail of the tensor-core attention kernels' arguments: cap, sink, gate pointer, gate pitch and, where
-    ``keep_first`` is given (a number), the learned sink's logits and the count of first keys that stay visible."""
+def _softmax_options(q, gate, num_heads, v_head_dim, softcap, sink, keep_first, slopes):
+    """The tail of the tensor-core attention kernels' arguments: cap, sink, gate pointer, gate pitch, the learned
+    sink's logits, the count of first keys that stay visible, and the distance bias's slopes."""
     if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1 or gate.dtype != q.dtype
                              or gate.shape[1] != num_heads * v_head_dim):
         raise ValueError("gate must be a matrix [tokens, heads * value size] of q's dtype with contiguous rows")
-    tail = (float(softcap or 0.0), _has_sink(sink), gate.data_ptr() if gate is not None else None,
-            gate.stride(0) if gate is not None else 0)
-    if keep_first is None:
-        if isinstance(sink, torch.Tensor):
-            raise ValueError("this kernel takes no learned sink")
-        return tail
-    return tail + (_sink_logits(sink, num_heads), int(keep_first))
+    return (float(softcap or 0.0), _has_sink(sink), gate.data_ptr() if gate is not None else None,
+            gate.stride(0) if gate is not None else 0, _sink_logits(sink, num_heads), int(keep_first),
+            _slopes_ptr(slopes, num_heads))
 
 
 def attn_decode_value_dim_supported(v_head_dim: int) -> bool:
@@ -1026,12 +1105,12 @@ def attn_decode_value_dim_supported(v_head_dim: int) -> bool:
 
 def attn_decode(q, cache, table, seq_rows, token_seq, positions, out, *, num_heads, num_kv_heads, head_dim, page_size,
                 scale, window=None, max_keys: int, num_pages=None, step_inputs_settled: bool = False, v_head_dim=None,
-                softcap=None, sink=False, gate=None, keep_first: int = 0):
+                softcap=None, sink=False, gate=None, keep_first: int = 0, slopes=None):
     """``step_inputs_settled``: ``table``, ``seq_rows``, ``token_seq`` and ``positions`` were complete
     before the kernel launched just before this call began (that kernel wrote ``q`` and the step's
     keys).  The attention kernel, launched as its dependent, then finds its place in the block table
-    while it still runs; otherwise it waits for it first.  ``v_head_dim``, ``softcap``, ``sink`` and
-    ``gate`` as :func:`paged_attention_plain`'s."""
+    while it still runs; otherwise it waits for it first.  ``v_head_dim``, ``softcap``, ``sink``,
+    ``gate`` and ``slopes`` as :func:`paged_attention_plain`'s."""
     tokens = q.shape[0]
     dv = int(v_head_dim or head_dim)
     splits, per = attn_decode_plan(tokens, num_heads, num_kv_heads, max_keys, sms=sm_count(q.device))
@@ -1039,28 +1118,28 @@ def attn_decode(q, cache, table, seq_rows, token_seq, positions, out, *, num_hea
     if splits > 1:
         part_o = torch.empty(tokens * num_heads * splits * dv, dtype=torch.float32, device=q.device)
         part_ml = torch.empty(tokens * num_heads * splits * 2, dtype=torch.float32, device=q.device)
-    _check(_fn("se_attn_decode", "pppipppppp" "iiiiii" "f" "iii" "ip" "i" "fipi" "pi" "p")(
+    _check(_fn("se_attn_decode", "pppipppppp" "iiiiii" "f" "iii" "ip" "i" "fipi" "pip" "p")(
         _ptr(q, torch.bfloat16, "q"), _ptr(cache, torch.bfloat16, "cache"), _ptr(table, torch.int32, "table"),
         table.shape[1], _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(token_seq, torch.int32, "token_seq"),
         _ptr(positions, torch.int32, "positions"), _ptr(out, torch.bfloat16, "out"), _ptr(part_o), _ptr(part_ml),
         tokens, num_heads, num_kv_heads, head_dim, dv, page_size, float(scale), int(window or 0), splits, per,
         cache.shape[0] if num_pages is None else int(num_pages), _ptr(error_word(q.device)),
-        int(bool(step_inputs_settled)), *_softmax_options(q, gate, num_heads, dv, softcap, sink, keep_first or 0),
+        int(bool(step_inputs_settled)), *_softmax_options(q, gate, num_heads, dv, softcap, sink, keep_first or 0, slopes),
         _stream()), "attn_decode")
     return out
 
 
 def attn_prefill(q, cache, table, seq_rows, cu_q, kv_len, out, *, entries, max_q_len, num_heads, num_kv_heads,
                  head_dim, page_size, scale, window=None, num_pages=None, v_head_dim=None, softcap=None,
-                 sink=False, gate=None, keep_first: int = 0):
+                 sink=False, gate=None, keep_first: int = 0, slopes=None):
     dv = int(v_head_dim or head_dim)
-    _check(_fn("se_attn_prefill", "pppipppp" "iiiiiii" "f" "i" "ip" "fipi" "pi" "p")(
+    _check(_fn("se_attn_prefill", "pppipppp" "iiiiiii" "f" "i" "ip" "fipi" "pip" "p")(
         _ptr(q, torch.bfloat16, "q"), _ptr(cache, torch.bfloat16, "cache"), _ptr(table, torch.int32, "table"),
         table.shape[1], _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(cu_q, torch.int32, "cu_q"),
         _ptr(kv_len, torch.int32, "kv_len"), _ptr(out, torch.bfloat16, "out"), entries, max_q_len, num_heads,
         num_kv_heads, head_dim, dv, page_size, float(scale), int(window or 0),
         cache.shape[0] if num_pages is None else int(num_pages), _ptr(error_word(q.device)),
-        *_softmax_options(q, gate, num_heads, dv, softcap, sink, keep_first or 0), _stream()), "attn_prefill")
+        *_softmax_options(q, gate, num_heads, dv, softcap, sink, keep_first or 0, slopes), _stream()), "attn_prefill")
     return out
 
 
@@ -1071,17 +1150,17 @@ def attn_prefill_tc_supported(head_dim: int, num_heads: int, num_kv_heads: int) 
 
 def attn_prefill_tc(q, cache, table, seq_rows, cu_q, kv_len, out, *, entries, max_q_len, num_heads, num_kv_heads,
                     head_dim, page_size, scale, window=None, num_pages=None, v_head_dim=None, softcap=None,
-                    sink: bool = False, gate=None, keep_first: int = 0):
+                    sink: bool = False, gate=None, keep_first: int = 0, slopes=None):
     """Prompt-portion attention on tcgen05 (head size 128, values of the same size)."""
     if int(v_head_dim or head_dim) != head_dim:
         raise ValueError("the tcgen05 prompt kernel takes values of the keys' head size")
-    _check(_fn("se_attn_prefill_tc", "pppippppp" "iiiiii" "f" "ii" "fipi" "pi" "p")(
+    _check(_fn("se_attn_prefill_tc", "pppippppp" "iiiiii" "f" "ii" "fipi" "pip" "p")(
         _ptr(q, torch.bfloat16, "q"), _ptr(cache, torch.bfloat16, "cache"), _ptr(table, torch.int32, "table"),
         table.shape[1], _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(cu_q, torch.int32, "cu_q"),
         _ptr(kv_len, torch.int32, "kv_len"), _ptr(out, torch.bfloat16, "out"), _ptr(error_word(q.device)),
         entries, max_q_len, num_heads, num_kv_heads, head_dim, page_size, float(scale), int(window or 0),
         cache.shape[0] if num_pages is None else int(num_pages),
-        *_softmax_options(q, gate, num_heads, head_dim, softcap, sink, keep_first or 0), _stream()),
+        *_softmax_options(q, gate, num_heads, head_dim, softcap, sink, keep_first or 0, slopes), _stream()),
         "attn_prefill_tc")
     return out
 

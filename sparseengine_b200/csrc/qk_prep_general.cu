@@ -11,8 +11,9 @@
 //              (u, v) -> (u cos a - v sin a, v cos a + u sin a), a = pos * inv_freq[i]  (rotary_dim = 0: none)
 //
 // Options: `bias` (32-bit, [q | k | v] like the projection row) is added to the projection before
-// anything else; `per_head` norms every head by its own root mean square, with weights of d elements
-// shared by the heads, instead of the whole projection with a weight per column.
+// anything else; `per_head` 1 norms every head by its own root mean square, with weights of d elements
+// shared by the heads, instead of the whole projection with a weight per column; `per_head` 2 does so for
+// queries and keys without weights.
 //
 // Everything is computed in 32-bit and rounded once.  The norm weights are
 // optional.  The projection row is [q: hq*d | k: hkv*d | v: hkv*dv] (`has_kv`) or [q] alone.
@@ -90,13 +91,14 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
         for (int h = warp; h < heads; h += warps) {
             const bool is_q = h < hq;
             float ss = 0.f;
-            if ((is_q ? q_w : k_w) != nullptr) {
+            const bool normed = per_head == 2 || (is_q ? q_w : k_w) != nullptr;
+            if (normed) {
                 const T* part = is_q ? row + (size_t)h * d : row + qn + (size_t)(h - hq) * d;
                 const int b0 = is_q ? h * d : qn + (h - hq) * d;
                 for (int i = lane; i < d; i += 32) { const float v = raw(part, b0, i); ss += v * v; }
                 ss = warp_sum(ss);
             }
-            if (lane == 0) inv_head[h] = (is_q ? q_w : k_w) != nullptr ? 1.0f / sqrtf(ss / (float)d + eps) : 1.f;
+            if (lane == 0) inv_head[h] = normed ? 1.0f / sqrtf(ss / (float)d + eps) : 1.f;
         }
         __syncthreads();
     } else {

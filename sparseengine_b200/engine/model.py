@@ -78,7 +78,13 @@ class Model:
                                       and all(b.mixer_streams.spec.streams == spec.streams for b in self.blocks)):
             raise ValueError("stream_mix blocks need residual_stream='float32', ModelSpec.streams equal to every block's, "
                              "an RMS final norm with a 32-bit weight, and no other arrangement beside them")
-        self.reinject = None
+        if not self.pending_stream and any(getattr(n.spec, "groups", 1) != 1 for n in self._norms()):
+            raise ValueError("norms in groups need pre_norm_stream blocks")
+        self.reinject = self.steps = None
+        if any(e.add_embedding or e.step_vector is not None for e in spec.order) and not self.pending_stream:
+            raise ValueError("ScheduleEntry.add_embedding and step_vector need pre_norm_stream blocks")
+        if any(e.step_vector is not None and not (spec.step_source and 0 <= e.step_vector < spec.step_count) for e in spec.order):
+            raise ValueError("ScheduleEntry.step_vector names a row of ModelSpec.step_source")
         if any(e.reinject for e in spec.order) and not (self.pending_stream and spec.reinject_source):
             raise ValueError("ScheduleEntry.reinject needs pre_norm_stream blocks and ModelSpec.reinject_source")
         for i, e in enumerate(spec.order):
@@ -87,6 +93,10 @@ class Model:
             if e.cache is not None and not 0 <= e.cache < i:
                 raise ValueError(f"schedule entry {i} reads the cache of entry {e.cache}, which is not earlier")
         self.layout = self._cache_layout()
+
+    def _norms(self) -> list:
+        parts = [p for b in self.blocks for name, p in b.parts().items() if name.endswith("norm")]
+        return parts + [self.final_norm]
 
     # ---- parameters --------------------------------------------------------------------
     def params(self) -> list[Param]:
@@ -98,6 +108,9 @@ class Model:
         if s.reinject_source is not None:
             out.append(Param(self, "reinject", "reinject", ParamSpec((s.hidden_size, 2 * s.hidden_size)),
                              (Source(s.reinject_source),)))
+        if s.step_source is not None:
+            out.append(Param(self, "steps", "steps", ParamSpec((s.step_count, s.hidden_size), "float32", "bias"),
+                             (Source(s.step_source),)))
         for name, p in self.final_norm.parameters().items():
             source = (s.final_norm_sources or {}).get(name, s.final_norm_source)
             out.append(Param(self.final_norm, name, f"final_norm.{name}", p, (Source(source),)))
@@ -166,8 +179,8 @@ class Model:
             entries.append(EntryCache(group, layer, write if kv is not None else False, state))
         return CacheLayout(tuple((g[0], g[1]) for g in groups), tuple(states), tuple(entries))
 
-    def _timed_block(self, block, hidden, residual, step, slot):
-        """The pre-norm block part by part with a CUDA event pair around each part."""
+    def _timed_block(self, block, hidden, residual, step, slot, inject=None):
+        """The block part by part with a CUDA event pair around each part."""
         def timed(name, fn, *a):
             e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             e0.record()
@@ -177,6 +190,8 @@ class Model:
             return out
         if isinstance(block, StreamMixBlock):
             return block.forward(hidden, residual, step, slot, timed=timed)
+        if isinstance(block, PreNormStreamBlock):
+            return block.forward(hidden, residual, step, slot, inject=inject, timed=timed)
         if isinstance(block, PostNormBlock):
             y = timed("mixer." + block.mixer.spec.kind, block.mixer.forward, hidden, step, slot)
             hidden, residual = timed("mixer_norm", block.mixer_norm.forward_stream, residual, y, block.alpha)
@@ -190,13 +205,6 @@ class Model:
             if block.feed_forward is not None:
                 y = timed("feed_forward." + block.feed_forward.spec.kind, block.feed_forward.forward, hidden, step)
                 hidden, residual = timed("feed_forward_norm", block.feed_forward_norm.forward_into_stream, residual, y)
-            return hidden, residual
-        if isinstance(block, PreNormStreamBlock):
-            x, residual = timed("mixer_norm", block.mixer_norm.forward_stream, residual, hidden)
-            hidden = timed("mixer." + block.mixer.spec.kind, block.mixer.forward, x, step, slot)
-            if block.feed_forward is not None:
-                x, residual = timed("feed_forward_norm", block.feed_forward_norm.forward_stream, residual, hidden)
-                hidden = timed("feed_forward." + block.feed_forward.spec.kind, block.feed_forward.forward, x, step)
             return hidden, residual
         if not isinstance(block, PreNormBlock):
             return timed("block", block.forward, hidden, residual, step, slot)
@@ -221,10 +229,10 @@ class Model:
             ops.stream_embed(self.embed, step.token_ids, residual, scale=s.embed_scale)
             hidden = None
         elif pending_stream:
-            # (output not yet added, 32-bit stream); `hidden` keeps the embedding output for the re-injections
+            # (output not yet added with its factor, 32-bit stream); `hidden` keeps the embedding output for the re-injections
             residual = torch.empty(hidden.shape, dtype=torch.float32, device=hidden.device)
-            ops.embed_stream(self.embed, step.token_ids, residual, hidden if self.dtype != torch.float32 else None,
-                             scale=s.embed_scale)
+            ops.embed_stream(self.embed, step.token_ids, residual,
+                             hidden if self.reinject is not None and self.dtype != torch.float32 else None, scale=s.embed_scale)
             if self.reinject is not None:
                 x0 = hidden if self.dtype != torch.float32 else residual.clone()
             hidden = None
@@ -244,15 +252,23 @@ class Model:
             if entry.reinject:
                 # the stream becomes W_x x + W_0 x0 (32-bit sums; x rounded to the activation type for the product)
                 x = torch.empty(residual.shape, dtype=self.dtype, device=residual.device)
-                ops.add_rmsnorm_stream(residual, hidden, None, 0.0, out_act=x)
+                y, alpha = hidden or (None, 1.0)
+                ops.add_rmsnorm_stream(residual, y, None, 0.0, out_act=x, alpha=alpha)
                 if x0_term is None:
                     x0_term = linear32(x0, self._reinject_0)
                 residual = linear32(x, self._reinject_x).add_(x0_term)
                 hidden = None
-            if self.profile is None:
-                hidden, residual = block.forward(hidden, residual, step, slot)
+            inject = None
+            if entry.add_embedding or entry.step_vector is not None:
+                # the embedding output (looked up once more, exact) and the pass's vector join the stream in the block's first norm
+                table, ids = (self.embed, step.token_ids) if entry.add_embedding else (None, None)
+                inject = (table, ids, s.embed_scale, self.steps[entry.step_vector] if entry.step_vector is not None else None)
+            if self.profile is not None:
+                hidden, residual = self._timed_block(block, hidden, residual, step, slot, inject)
+            elif inject is not None:
+                hidden, residual = block.forward(hidden, residual, step, slot, inject=inject)
             else:
-                hidden, residual = self._timed_block(block, hidden, residual, step, slot)
+                hidden, residual = block.forward(hidden, residual, step, slot)
             if self.stream_taps is not None and self.multi_stream:
                 both = residual.clone()          # the streams with the result they have not taken in yet, as one
                 ops.stream_mix(both, write=hidden[0].write_args(hidden[1], hidden[2]), dtype=self.dtype)
@@ -261,7 +277,7 @@ class Model:
             elif self.stream_taps is not None:
                 tap = (residual if stream32 else hidden).float().clone()
                 if pending_stream and hidden is not None:
-                    tap += hidden.float()
+                    tap += hidden[0].float() * hidden[1]
                 self.stream_taps.append(tap)
         if want_rows is None or want_rows.numel() == 0:
             return None
@@ -283,11 +299,12 @@ class Model:
         elif pending_stream:  # the wanted rows of the stream and of what it has not taken in yet
             r = torch.empty(n, s.hidden_size, dtype=torch.float32, device=residual.device)
             ops.gather_rows(residual, want_rows, r)
-            p = None
+            p, alpha = None, 1.0
             if hidden is not None:
+                y, alpha = hidden
                 p = torch.empty(n, s.hidden_size, dtype=self.dtype, device=residual.device)
-                ops.gather_rows(hidden, want_rows, p)
-            h, _ = self.final_norm.forward_stream(r, p)
+                ops.gather_rows(y, want_rows, p)
+            h, _ = self.final_norm.forward_stream(r, p, alpha)
         elif stream32:      # the final norm reads the wanted rows of the stream
             r = torch.empty(n, s.hidden_size, dtype=torch.float32, device=hidden.device)
             ops.gather_rows(residual, want_rows, r)

@@ -8,8 +8,8 @@ written before attention reads the cache.
 The general preparation (``prep="general"``) adds, each by a field of the spec: values of a head
 size of their own, a query temperature, layers without keys of their own, a cap on the scores,
 a sink of score 0 or of a learned score per head in the softmax, an output gate, values blended with
-those of an earlier layer, norms per head, biases on the projections, and first positions that stay
-visible beside a window.  The blended values are what is cached; the earlier layer's values of this step's tokens
+those of an earlier layer, norms per head (with or without a weight), biases on the projections, a
+distance bias on the scores, and first positions that stay visible beside a window.  The blended values are what is cached; the earlier layer's values of this step's tokens
 travel from layer to layer in the step's scratch (``StepContext.extras``), so nothing of them
 is kept between steps.
 """
@@ -52,17 +52,19 @@ class PagedAttention(Mixer):
                 raise ValueError("q_temperature is (coef, every) with every > 0")
         elif (s.v_head_dim not in (None, s.head_dim) or s.q_temperature is not None or not s.own_kv
               or s.score_softcap is not None or s.sink is not None or s.output_gate or s.value_mix is not None
-              or s.bias or s.keep_first or s.qk_norm == "per_head"):
+              or s.bias or s.keep_first or s.distance_slopes is not None or s.qk_norm in ("per_head", "per_head_unit")):
             raise ValueError("v_head_dim, q_temperature, own_kv=False, score_softcap, sink, output_gate, value_mix, "
-                             "bias, keep_first and per-head norms need prep='general'")
+                             "bias, keep_first, distance_slopes and per-head norms need prep='general'")
         elif s.head_dim <= 0 or s.head_dim % 16 or s.head_dim > ops.LIMITS["attention_max_head_dim"]:
             raise ValueError(f"head_dim {s.head_dim} is not supported (multiples of 16 up to "
                              f"{ops.LIMITS['attention_max_head_dim']})")
         if s.num_heads > ops.LIMITS["grid_dim_yz"]:
             raise ValueError(f"{s.num_heads} query heads are not supported (at most {ops.LIMITS['grid_dim_yz']}: "
                              "heads are a grid dimension of the attention kernels)")
-        if s.qk_norm not in (None, "whole_projection", "per_head"):
-            raise ValueError(f"qk_norm {s.qk_norm!r} is not supported (None, 'whole_projection' or 'per_head')")
+        if s.qk_norm not in (None, "whole_projection", "per_head", "per_head_unit"):
+            raise ValueError(f"qk_norm {s.qk_norm!r} is not supported (None, 'whole_projection', 'per_head' or 'per_head_unit')")
+        if s.distance_slopes is not None and len(s.distance_slopes) != s.num_heads:
+            raise ValueError(f"distance_slopes needs one slope per query head ({s.num_heads}), got {len(s.distance_slopes)}")
         if s.keep_first < 0 or (s.keep_first and s.window is None):
             raise ValueError("keep_first is a count of first positions that stay visible beside a window")
         if s.bias and (s.output_gate or not s.own_kv):
@@ -82,6 +84,7 @@ class PagedAttention(Mixer):
         if rot > s.head_dim:
             raise ValueError(f"the position encoding rotates {rot} dims, a head has {s.head_dim}")
         self.q_norm = self.k_norm = self.v_mix = self.qkv_bias = self.o_bias = self.sink = None
+        self._slopes = None
         # True: whoever combines this mixer's output with others adds `o_bias` (see `output_bias`)
         self.defer_output_bias = False
 
@@ -94,7 +97,7 @@ class PagedAttention(Mixer):
         out = {"qkv": ParamSpec((rows, s.hidden_size)), "o": ParamSpec((s.hidden_size, s.num_heads * s.value_dim))}
         if s.value_mix is not None:
             out["v_mix"] = ParamSpec((), "float32", "unit")
-        if s.qk_norm is not None:
+        if s.qk_norm in ("whole_projection", "per_head"):
             per_head = s.qk_norm == "per_head"      # one weight of head_dim elements for all heads
             out["q_norm"] = ParamSpec((s.head_dim if per_head else q,), "act", "norm")
             if s.own_kv:
@@ -148,7 +151,7 @@ class PagedAttention(Mixer):
                             head_dim=s.head_dim, v_head_dim=s.value_dim, eps=s.qk_norm_eps, page_size=slot.page_size,
                             has_kv=writes, temperature=s.q_temperature, inv_freq=inv_freq, rotary_dim=rotary_dim,
                             v_first=v_first, v_mix=self.v_mix if v_first is not None else None, bias=self.qkv_bias,
-                            per_head=s.qk_norm == "per_head")
+                            per_head=s.qk_norm == "per_head", per_head_unit=s.qk_norm == "per_head_unit")
         attn = torch.empty(tokens, s.num_heads * s.value_dim, dtype=x.dtype, device=x.device)
         gate = None
         if s.output_gate:
@@ -203,7 +206,14 @@ class PagedAttention(Mixer):
             return True
         return (step.max_q_len >= self.portion_min_tokens
                 and step.num_tokens >= self.portion_min_average * step.num_seqs)
+
     use_tensor_cores = None      # False: always the plain kernel
+
+    def slopes(self, device):
+        """The distance bias's slopes on the device (32-bit), or None."""
+        if self.spec.distance_slopes is not None and (self._slopes is None or self._slopes.device != torch.device(device)):
+            self._slopes = torch.tensor([float(v) for v in self.spec.distance_slopes], dtype=torch.float32, device=device)
+        return self._slopes
 
     def attend(self, q, out, step, slot, after_qk_prep=False, gate=None):
         """``after_qk_prep``: the kernel launched last is the one that wrote this step's keys and
@@ -211,7 +221,8 @@ class PagedAttention(Mixer):
         ``gate``: the output gate's projection (a view with a row pitch), or None."""
         s = self.spec
         sink = self.sink if s.sink == "learned" else s.sink == "zero"
-        options = dict(v_head_dim=s.value_dim, softcap=s.score_softcap, sink=sink, gate=gate, keep_first=s.keep_first)
+        options = dict(v_head_dim=s.value_dim, softcap=s.score_softcap, sink=sink, gate=gate, keep_first=s.keep_first,
+                       slopes=self.slopes(q.device))
         if (self.use_tensor_cores is not False and q.dtype == torch.bfloat16
                 and ops.attn_decode_supported(s.head_dim, s.num_heads, s.num_kv_heads)
                 and ops.attn_decode_value_dim_supported(s.value_dim)):

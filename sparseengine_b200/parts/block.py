@@ -81,16 +81,18 @@ class PostNormBlock:
 
 
 class PreNormStreamBlock:
-    """Norm before each sublayer, over a 32-bit stream: ``x <- x + mixer(norm(x))``, then (if the layer
-    has a feed-forward) ``x <- x + feed_forward(norm(x))``.  The block carries ``(pending, stream)``:
-    ``pending`` is the last sublayer's output that the stream has not taken in yet (None at the
-    start); the next norm call adds it in 32-bit and normalises the sum in one kernel.  Whoever
-    needs the stream itself (the model's last norm, a tap, the start of a looped pass) adds
-    ``pending`` first.  The norms are parts with ``forward_stream(stream, y)``
-    (``parts.norm.RMSNorm``)."""
+    """Norm before each sublayer, over a 32-bit stream: ``x <- x + a * mixer(norm(x))``, then (if the layer
+    has a feed-forward) ``x <- x + a * feed_forward(norm(x))`` with ``a = residual_scale``.  The block carries
+    ``(pending, stream)``: ``pending = (y, a)`` is the last sublayer's output that the stream has not
+    taken in yet, with its factor (None at the start); the next norm call adds it in 32-bit and
+    normalises the sum in one kernel.  Whoever needs the stream itself (the model's last norm, a tap,
+    the start of a looped pass) adds ``pending`` first.  ``inject``: what else joins the stream ahead of
+    the block's first norm, in the same kernel (``ops.add_rmsnorm_stream``).  The norms are parts with
+    ``forward_stream(stream, y, alpha, inject)`` (``parts.norm.RMSNorm``)."""
 
     def __init__(self, spec, dtype):
         self.spec = spec
+        self.alpha = float(spec.residual_scale)
         self.mixer = make_mixer(spec.mixer, dtype)
         self.mixer_norm = make_norm(spec.mixer_norm, dtype)
         self.feed_forward = self.feed_forward_norm = None
@@ -108,13 +110,14 @@ class PreNormStreamBlock:
             out["feed_forward_norm"] = self.feed_forward_norm
         return out
 
-    def forward(self, pending, stream, step, slot):
-        x, stream = self.mixer_norm.forward_stream(stream, pending)
-        pending = self.mixer.forward(x, step, slot)
+    def forward(self, pending, stream, step, slot, inject=None, timed=None):
+        run = timed if timed is not None else (lambda name, fn, *a: fn(*a))
+        x, stream = run("mixer_norm", self.mixer_norm.forward_stream, stream, *(pending or (None, 1.0)), inject)
+        y = run("mixer." + self.mixer.spec.kind, self.mixer.forward, x, step, slot)
         if self.feed_forward is not None:
-            x, stream = self.feed_forward_norm.forward_stream(stream, pending)
-            pending = self.feed_forward.forward(x, step)
-        return pending, stream
+            x, stream = run("feed_forward_norm", self.feed_forward_norm.forward_stream, stream, y, self.alpha)
+            y = run("feed_forward." + self.feed_forward.spec.kind, self.feed_forward.forward, x, step)
+        return (y, self.alpha), stream
 
 
 class SublayerNormBlock:

@@ -3,7 +3,8 @@
 Per token the mixer projects to ``[query latent | key/value latent | shared rotated key part]`` in
 one product; the preparation kernel RMS-norms the two latents (32-bit), rotates the shared key
 part and writes ``[c | k_rot]`` into the token's page slot: that row is all the cache holds.
-Queries ``q = W_uq c_q`` are laid out head by head as ``[head_dim unrotated | rot_dim rotated]``.
+Queries ``q = W_uq c_q`` (or, without a query latent, ``q = W_q x``: the one product is then ``[queries |
+key/value latent | shared rotated key part | output gate]`` and the kernels read its columns) are laid out head by head as ``[head_dim unrotated | rot_dim rotated]``.
 
 Keys and values are never formed.  With ``k_plain = W_uk c`` and ``v = W_uv c``,
 
@@ -23,7 +24,7 @@ from ..config.specs import ParamSpec
 from ..csrc import ops
 from .base import KVRequest, Mixer, make_position, register_mixer
 from .linear import linear
-from .position import as_rotary_args
+from .position import RotaryArgs, as_rotary_args
 
 
 class LatentAttention(Mixer):
@@ -33,8 +34,10 @@ class LatentAttention(Mixer):
     def __init__(self, spec, dtype):
         super().__init__(spec, dtype)
         s = spec
-        if min(s.hidden_size, s.num_heads, s.head_dim, s.v_head_dim, s.q_rank, s.kv_rank) <= 0 or s.rot_dim < 0:
-            raise ValueError("the sizes of a latent attention must be positive (rot_dim may be 0)")
+        if min(s.hidden_size, s.num_heads, s.head_dim, s.v_head_dim, s.kv_rank) <= 0 or s.rot_dim < 0 or s.q_rank < 0:
+            raise ValueError("the sizes of a latent attention must be positive (rot_dim and q_rank may be 0)")
+        if s.output_gate and s.q_rank:
+            raise ValueError("an output gate goes with queries straight from the input (q_rank 0)")
         if s.kv_rank + s.rot_dim > ops.LIMITS["latent_max_row"]:
             raise ValueError(f"a cached row of {s.kv_rank} + {s.rot_dim} elements is not supported (at most "
                              f"{ops.LIMITS['latent_max_row']}: a warp keeps a row in registers)")
@@ -44,18 +47,25 @@ class LatentAttention(Mixer):
             raise ValueError("window must be positive (None: all keys)")
         self.position = make_position(s.position, dtype) if s.position is not None and s.rot_dim > 0 else None
         if self.position is not None:
-            if s.position.pairing != "split_half":
-                raise ValueError("the latent attention kernels rotate split halves only")
+            if s.position.pairing not in ("split_half", "interleaved"):
+                raise ValueError("the latent attention kernels rotate split halves or interleaved pairs")
             if s.position.rotary_dim > s.rot_dim:
                 raise ValueError(f"the position encoding rotates {s.position.rotary_dim} dims, the rotated part has {s.rot_dim}")
         self.sink = None
+        # without a query latent: the columns of the one projection
+        self.q_cols = 0 if s.q_rank else s.num_heads * (s.head_dim + s.rot_dim)
+        self.g_off = self.q_cols + s.kv_rank + s.rot_dim
+        self.g_cols = s.num_heads * s.v_head_dim if s.output_gate else 0
 
     def parameters(self):
         s = self.spec
-        out = {"down": ParamSpec((s.q_rank + s.kv_rank + s.rot_dim, s.hidden_size)),
-               "q_norm": ParamSpec((s.q_rank,), "act", "norm"),
-               "kv_norm": ParamSpec((s.kv_rank,), "act", "norm"),
-               "uq": ParamSpec((s.num_heads * (s.head_dim + s.rot_dim), s.q_rank)),
+        if s.q_rank:
+            out = {"down": ParamSpec((s.q_rank + s.kv_rank + s.rot_dim, s.hidden_size)),
+                   "q_norm": ParamSpec((s.q_rank,), "act", "norm"),
+                   "uq": ParamSpec((s.num_heads * (s.head_dim + s.rot_dim), s.q_rank))}
+        else:       # queries, then what `down` holds, then the gate
+            out = {"in_proj": ParamSpec((self.g_off + self.g_cols, s.hidden_size))}
+        out |= {"kv_norm": ParamSpec((s.kv_rank,), "act", "norm"),
                "uk": ParamSpec((s.num_heads * s.head_dim, s.kv_rank)),
                "uv": ParamSpec((s.num_heads * s.v_head_dim, s.kv_rank)),
                "o": ParamSpec((s.hidden_size, s.num_heads * s.v_head_dim))}
@@ -75,29 +85,32 @@ class LatentAttention(Mixer):
             rope = as_rotary_args(self.position.kernel_args(dev))
             if rope.scale != 1.0:
                 raise ValueError("the latent attention kernels take no factor on cos and sin")
-            inv_freq, rotary_dim = rope.inv_freq, rope.rotary_dim
         else:
-            inv_freq, rotary_dim = None, 0
-        proj = linear(x, self.down)
-        cq = torch.empty(tokens, s.q_rank, dtype=x.dtype, device=dev)
-        ops.latent_prep(proj, self.q_norm, self.kv_norm, inv_freq, step.positions, step.token_seq, step.seq_rows,
-                        slot.table, slot.kv, cq, q_rank=s.q_rank, rank=rank, rot=r, rotary_dim=rotary_dim,
-                        eps=s.norm_eps, page_size=slot.page_size, write_cache=slot.write_cache)
-        q = linear(cq, self.uq)                                              # [tokens, H * (d + r)]
+            rope = RotaryArgs(None, 0)
+        proj = linear(x, self.down if s.q_rank else self.in_proj)
+        cq = torch.empty(tokens, s.q_rank, dtype=x.dtype, device=dev) if s.q_rank else None
+        ops.latent_prep(proj[:, self.q_cols:self.g_off + s.q_rank], self.q_norm if s.q_rank else None, self.kv_norm,
+                        rope.inv_freq, step.positions, step.token_seq, step.seq_rows, slot.table, slot.kv, cq,
+                        q_rank=s.q_rank, rank=rank, rot=r, rotary_dim=rope.rotary_dim, eps=s.norm_eps,
+                        page_size=slot.page_size, write_cache=slot.write_cache, pairing=rope.pairing)
+        q = linear(cq, self.uq) if s.q_rank else proj[:, :self.q_cols]       # [tokens, H * (d + r)]
         # the unrotated queries in the latent's space: [H, tokens, d] x [H, d, rank], 32-bit out
-        q_plain = q.view(tokens, H, d + r)[:, :, :d].transpose(0, 1)
+        q_plain = q.unflatten(1, (H, d + r))[:, :, :d].transpose(0, 1)
         q_lat = torch.bmm(q_plain, self.uk.view(H, d, rank), out_dtype=torch.float32) if x.dtype != torch.float32 \
             else torch.bmm(q_plain, self.uk.view(H, d, rank))
         out_lat = torch.empty(tokens, H, rank, dtype=x.dtype, device=dev)
-        self.attend(q_lat, q, inv_freq, rotary_dim, out_lat, step, slot)
+        self.attend(q_lat, q, rope, out_lat, step, slot)
         # the values' up-projection per head, read from and written to token-major rows through strided views
         heads_out = torch.empty(tokens, H, s.v_head_dim, dtype=x.dtype, device=dev)
         torch.bmm(out_lat.transpose(0, 1), self.uv.view(H, s.v_head_dim, rank).transpose(1, 2), out=heads_out.transpose(0, 1))
-        return linear(heads_out.view(tokens, H * s.v_head_dim), self.o)
+        heads_out = heads_out.view(tokens, H * s.v_head_dim)
+        if s.output_gate:
+            ops.sigmoid_gate_(heads_out, proj[:, self.g_off:])
+        return linear(heads_out, self.o)
 
     use_tensor_cores = None      # False: always the kernel with one block per (token, head)
 
-    def attend(self, q_lat, q, inv_freq, rotary_dim, out_lat, step, slot):
+    def attend(self, q_lat, q, rope, out_lat, step, slot):
         """bfloat16 steps of sizes the tiled kernel takes (latent and rotated part in multiples of 16, a
         cached row of at most 256) run on tensor-core tiles whose rows are (token, head) pairs, prompt
         portions and single tokens alike; everything else one block per (token, head)."""
@@ -105,18 +118,18 @@ class LatentAttention(Mixer):
         if (self.use_tensor_cores is not False and q.dtype == torch.bfloat16 and s.scale > 0
                 and ops.latent_attention_tiled_supported(s.kv_rank, s.rot_dim)):
             qfull = torch.empty(q.shape[0], s.num_heads, s.kv_rank + s.rot_dim, dtype=q.dtype, device=q.device)
-            ops.latent_q_pack(q_lat, q, inv_freq, step.positions, qfull, heads=s.num_heads, head_dim=s.head_dim,
-                              rank=s.kv_rank, rot=s.rot_dim, rotary_dim=rotary_dim)
+            ops.latent_q_pack(q_lat, q, rope.inv_freq, step.positions, qfull, heads=s.num_heads, head_dim=s.head_dim,
+                              rank=s.kv_rank, rot=s.rot_dim, rotary_dim=rope.rotary_dim, pairing=rope.pairing)
             ops.latent_attention_tiled(qfull, slot.kv, slot.table, step.seq_rows, step.cu_q, step.kv_len, self.sink,
                                        out_lat, entries=step.num_seqs, max_q_len=step.max_q_len, heads=s.num_heads,
                                        rank=s.kv_rank, rot=s.rot_dim, page_size=slot.page_size, scale=s.scale,
                                        window=s.window,
                                        max_keys=step.max_kv_len if s.window is None else min(step.max_kv_len, s.window + step.max_q_len - 1))
             return
-        ops.latent_attention_plain(q_lat, q, inv_freq, slot.kv, slot.table, step.seq_rows, step.token_seq,
+        ops.latent_attention_plain(q_lat, q, rope.inv_freq, slot.kv, slot.table, step.seq_rows, step.token_seq,
                                    step.positions, self.sink, out_lat, heads=s.num_heads, head_dim=s.head_dim,
-                                   rank=s.kv_rank, rot=s.rot_dim, rotary_dim=rotary_dim, page_size=slot.page_size,
-                                   scale=s.scale, window=s.window)
+                                   rank=s.kv_rank, rot=s.rot_dim, rotary_dim=rope.rotary_dim, page_size=slot.page_size,
+                                   scale=s.scale, window=s.window, pairing=rope.pairing)
 
 
 register_mixer("latent_attention", LatentAttention)

@@ -21,6 +21,13 @@ class RMSNorm(Norm):
                              f"{ops.LIMITS['rmsnorm_max_width']} elements")
         if not spec.eps > 0:
             raise ValueError("RMSNorm eps must be positive")
+        if spec.groups < 1 or spec.size % spec.groups or spec.groups > ops.LIMITS["rmsnorm_stream_max_groups"]:
+            raise ValueError(f"{spec.groups} groups do not divide a norm of width {spec.size} (or are more than "
+                             f"{ops.LIMITS['rmsnorm_stream_max_groups']})")
+
+    def _whole_rows_only(self):
+        if self.spec.groups != 1:
+            raise ValueError("a norm in groups works on a 32-bit pre-norm stream only (forward_stream)")
 
     def parameters(self):
         if self.spec.offset:        # kept in 32-bit: offset + w would lose the stored digits in a 16-bit type
@@ -33,6 +40,7 @@ class RMSNorm(Norm):
             self.weight = self.weight + float(self.spec.offset)     # what the kernels multiply by
 
     def forward(self, x, residual=None):
+        self._whole_rows_only()
         out = torch.empty_like(x)
         if residual is None:
             ops.rmsnorm(x, self.weight, self.spec.eps, out)
@@ -41,18 +49,21 @@ class RMSNorm(Norm):
         ops.rmsnorm(x, self.weight, self.spec.eps, out, residual=residual, residual_out=new_residual)
         return out, new_residual
 
-    def forward_stream(self, stream, y=None):
-        """Over a 32-bit residual stream (kernel: csrc/stream32.cu): ``stream += y`` in place (``y``:
+    def forward_stream(self, stream, y=None, alpha: float = 1.0, inject=None):
+        """Over a 32-bit residual stream (kernel: csrc/stream32.cu): ``stream += alpha * y`` in place (``y``:
         the last sublayer's output in the activation type, or None), then the norm of the sum in the
-        activation type.  Returns ``(normed, stream)``."""
+        activation type.  ``inject``: what else joins the stream (``ops.add_rmsnorm_stream``).  Returns
+        ``(normed, stream)``."""
         out = torch.empty(stream.shape, dtype=self.dtype, device=stream.device)
-        ops.add_rmsnorm_stream(stream, y, self.weight, self.spec.eps, out32=stream if y is not None else None, out_act=out)
+        ops.add_rmsnorm_stream(stream, y, self.weight, self.spec.eps, out32=stream if y is not None or inject is not None else None,
+                               out_act=out, alpha=alpha, groups=self.spec.groups, inject=inject)
         return out, stream
 
     def forward_into_stream(self, stream, y):
         """A norm on a sublayer's output (kernel: csrc/stream32.cu): ``stream += norm(y)`` in place
         (32-bit).  Returns ``(the new stream in the activation type, stream)``; in a 32-bit engine the
         first is the stream itself."""
+        self._whole_rows_only()
         if self.dtype == torch.float32:
             ops.rmsnorm_add_stream(stream, y, self.weight, self.spec.eps)
             return stream, stream

@@ -292,6 +292,41 @@ class MatrixMemoryMixer(Mixer):
         return linear(gated, self.o)
 
 
+class MinGRUMixer(Mixer):
+    """``[z | x | g] = in_proj(h)``; a gated running average per channel (``config.specs.MinGRUSpec``; kernels:
+    csrc/min_gru.cu).  The state is one 32-bit row of ``width`` numbers per request."""
+    graph_safe = True
+    chunk_min_tokens = 8         # the longest entry of a step from which the chunked kernel runs; None: never
+
+    def __init__(self, spec, dtype):
+        super().__init__(spec, dtype)
+        if min(spec.width, spec.hidden_size) <= 0:
+            raise ValueError("the sizes of a minGRU mixer must be positive")
+        if -(-spec.width // 64) > ops.LIMITS["grid_dim_yz"]:
+            raise ValueError(f"width {spec.width} is not supported (groups of 64 channels are a grid dimension of the kernels)")
+
+    max_step_entries = ops.LIMITS["grid_dim_yz"]
+
+    def parameters(self):
+        s = self.spec
+        return {"in_proj": ParamSpec((3 * s.width, s.hidden_size)),
+                "gate_bias": ParamSpec((2 * s.width,), "float32", "bias"),      # of z, then of x
+                "o": ParamSpec((s.hidden_size, s.width))}
+
+    def state_request(self):
+        return StateRequest((self.spec.width,), torch.float32)
+
+    def forward(self, x, step, slot):
+        proj = linear(x, self.in_proj)
+        y = torch.empty(x.shape[0], self.spec.width, dtype=x.dtype, device=x.device)
+        # a step with a prompt portion deals a request's tokens out to many warps; steps of single tokens and of
+        # short pieces walk them
+        chunked = self.chunk_min_tokens is not None and step.max_q_len >= self.chunk_min_tokens
+        (ops.min_gru_chunk if chunked else ops.min_gru_scan)(proj, self.gate_bias, slot.state, step, y)
+        return linear(y, self.o)
+
+
+register_mixer("mingru", MinGRUMixer)
 register_mixer("matrix_memory", MatrixMemoryMixer)
 register_mixer("retention", RetentionMixer)
 register_mixer("mamba2", StateSpaceMixer)
