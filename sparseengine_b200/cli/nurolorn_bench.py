@@ -109,22 +109,19 @@ def _kernels(width: int, cases, pk: dict) -> dict:
         kw = torch.ones(rank, device=dev, dtype=bf)
         inv = (1e6 ** (-torch.arange(0, r, 2, dtype=torch.float32) / r)).to(dev)
         cq, qw = torch.empty(tokens, width // 2, device=dev, dtype=bf), torch.ones(width // 2, device=dev, dtype=bf)
-        add("latent_prep (no query latent, neighbouring pairs)", lambda: ops.latent_prep(
+        qfull = torch.zeros(tokens, H, D, device=dev, dtype=bf)
+        add("latent_prep (no query latent, neighbouring pairs, queries)", lambda: ops.latent_prep(
             proj[:, cols:cols + D], None, kw, inv, step.positions, step.token_seq, step.seq_rows, btable, cache, None, q_rank=0,
-            rank=rank, rot=r, rotary_dim=r, eps=1e-6, page_size=PAGE_SIZE, pairing="interleaved"), tokens * D * 4)
+            rank=rank, rot=r, rotary_dim=r, eps=1e-6, page_size=PAGE_SIZE, pairing="interleaved",
+            queries=(proj[:, :cols], H, d, qfull)), tokens * (D + H * r) * 4)
         proj_q = torch.randn(tokens, width // 2 + D, device=dev, dtype=bf)
         add("like: latent_prep (query latent, split halves)", lambda: ops.latent_prep(
             proj_q, qw, kw, inv, step.positions, step.token_seq, step.seq_rows, btable, cache, cq, q_rank=width // 2, rank=rank,
             rot=r, rotary_dim=r, eps=1e-6, page_size=PAGE_SIZE), tokens * (width // 2 + D) * 4)
-        q_lat = torch.randn(H, tokens, rank, device=dev)
-        qfull = torch.empty(tokens, H, D, device=dev, dtype=bf)
-        pack_bytes = tokens * H * (rank * 4 + r * 2 + D * 2)
-        add("latent_q_pack (neighbouring pairs)", lambda: ops.latent_q_pack(
-            q_lat, proj[:, :cols], inv, step.positions, qfull, heads=H, head_dim=d, rank=rank, rot=r, rotary_dim=r,
-            pairing="interleaved"), pack_bytes)
         q = torch.randn(tokens, cols, device=dev, dtype=bf)
-        add("like: latent_q_pack (split halves)", lambda: ops.latent_q_pack(
-            q_lat, q, inv, step.positions, qfull, heads=H, head_dim=d, rank=rank, rot=r, rotary_dim=r), pack_bytes)
+        add("like: latent_q_rotate (split halves)", lambda: ops.latent_q_rotate(
+            q, inv, step.positions, qfull, heads=H, head_dim=d, rank=rank, rot=r, rotary_dim=r), tokens * H * r * 4)
+        qfull[:, :, :rank].normal_()
         o_lat = torch.empty(tokens, H, rank, device=dev, dtype=bf)
 
         def tiled(window, sink):

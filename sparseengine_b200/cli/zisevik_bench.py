@@ -98,8 +98,8 @@ def _kernels(width: int, cases, pk: dict) -> dict:
         q = torch.randn(tokens, H * (d + r), device=dev, dtype=bf)
         q_lat = torch.randn(H, tokens, rank, device=dev)
         qfull = torch.empty(tokens, H, D, device=dev, dtype=bf)
-        add("latent_q_pack", lambda: ops.latent_q_pack(q_lat, q, inv, step.positions, qfull, heads=H, head_dim=d, rank=rank, rot=r,
-                                                       rotary_dim=r), tokens * H * (rank * 4 + r * 2 + D * 2))
+        add("latent_q_rotate", lambda: ops.latent_q_rotate(q, inv, step.positions, qfull, heads=H, head_dim=d, rank=rank, rot=r,
+                                                           rotary_dim=r), tokens * H * r * 4)
         sink = torch.zeros(H, device=dev)
         o_lat = torch.empty(tokens, H, rank, device=dev, dtype=bf)
         # keys a query sees: min(window, position + 1)

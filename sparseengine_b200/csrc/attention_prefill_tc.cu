@@ -355,16 +355,13 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             }
             const bool first = j < kept_tiles;
             const int key0 = first ? j * kKeys : k_begin + (j - kept_tiles) * kKeys;
+            // the distance bias slope * (key - pos): its part within the tile joins the scores here, the tile's first
+            // key's (log2 units) joins the maximum and the exponents below
+            float tile_bias = 0.f;
             if (opt.slopes != nullptr) {
-                // s + slope * (key - pos), two keys at a time (differences of positions are exact in 32-bit)
-                float2* s2 = reinterpret_cast<float2*>(sv);
-                const float d0 = (float)(key0 - pos);
-                float2 d = make_float2(d0, d0 + 1.f);
+                tile_bias = slope * (float)(key0 - pos) * scale_log2;
 #pragma unroll
-                for (int c = 0; c < 32; ++c) {
-                    s2[c] = se::mma::fma2(make_float2(slope, slope), d, s2[c]);
-                    d.x += 2.f; d.y += 2.f;
-                }
+                for (int c = 1; c < 64; ++c) sv[c] = __float_as_uint(fmaf(slope, (float)c, __uint_as_float(sv[c])));
             }
             // A tile every row of the warp sees in full needs no masking (rows ascend with the
             // lane: lane 0 has the smallest position, lane 31 the largest window start).  A tile of kept first keys
@@ -389,7 +386,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                 m4[3] = fmaxf(m4[3], __uint_as_float(sv[c + 3]));
             }
             float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
-            mx *= scale_log2;                                            // log2 units (scale > 0)
+            mx = fmaf(mx, scale_log2, tile_bias);                        // log2 units (scale > 0)
             // move the reference maximum only on the first visible keys or a large jump
             float factor = 1.f;
             bool need = false;
@@ -418,7 +415,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             }
             const float m_use = m_ref == -INFINITY ? 0.f : m_ref;
             float sum4[4] = {0.f, 0.f, 0.f, 0.f};
-            const float neg_m = -m_use;
+            const float neg_m = tile_bias - m_use;
             // P goes back to tensor memory, over the row's own scores (which are in registers now):
             // two bfloat16 per column, the A operand of P·V.
             uint32_t packed[32];

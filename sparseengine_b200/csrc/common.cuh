@@ -159,4 +159,12 @@ template <typename T> __device__ __forceinline__ bool aligned8(const T* p) {
     return (reinterpret_cast<uintptr_t>(p) & 15) == 0;
 }
 
+// An ungated feed-forward's activation.
+__device__ __forceinline__ float act_apply(float v, int kind) {
+    if (kind == 0) { const float r = fmaxf(v, 0.f); return r * r; }                       // squared relu
+    if (kind == 1) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));   // gelu (tanh form)
+    if (kind == 2) return v / (1.f + expf(-v));                                           // silu
+    return fmaxf(v, 0.f);                                                                 // relu
+}
+
 }  // namespace se

@@ -30,7 +30,7 @@ namespace gemv {
 template <int NT, int kWarps, int kRowsPerBlock>
 __global__ void __launch_bounds__(32 * kWarps)
 gemv_kernel(const __nv_bfloat16* x, const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
-            int rows, int n_out, int k_dim) {
+            int rows, int n_out, int k_dim, int act) {
     grid_dependency_trigger();       // the kernel after this one may set itself up meanwhile
     constexpr int kPreload = SE_GEMV_PRELOAD;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -103,7 +103,9 @@ gemv_kernel(const __nv_bfloat16* x, const __nv_bfloat16* __restrict__ w, __nv_bf
             float v = 0.f;
 #pragma unroll
             for (int wq = 0; wq < kWarps; ++wq) v += part[wq][r][t];
-            out[(size_t)t * n_out + n0 + r] = __float2bfloat16_rn(v);
+            const __nv_bfloat16 y = __float2bfloat16_rn(v);
+            // as a product and an activation in two kernels would: the activation reads the rounded product
+            out[(size_t)t * n_out + n0 + r] = act >= 0 ? __float2bfloat16_rn(act_apply(__bfloat162float(y), act)) : y;
         }
     }
 }
@@ -116,14 +118,16 @@ extern "C" int se_gemv_supported(int rows, int n_out, int k_dim) {
 }
 
 template <int NT, int W, int R>
-static void launch_gemv(const void* x, const void* w, void* out, int rows, int n_out, int k_dim, cudaStream_t stream) {
+static void launch_gemv(const void* x, const void* w, void* out, int rows, int n_out, int k_dim, int act, cudaStream_t stream) {
     SE_LAUNCH_DEPENDENT("gemv", se::gemv::gemv_kernel<NT, W, R>, dim3(se::ceil_div(n_out, R)), dim3(32 * W), 0, stream,
-                         (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, rows, n_out, k_dim);
+                         (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, rows, n_out, k_dim, act);
 }
 
-// x [rows <= 16, k_dim], w [n_out, k_dim], out [rows, n_out]; bf16; k_dim a multiple of 32.
-extern "C" int se_gemv(const void* x, const void* w, void* out, int rows, int n_out, int k_dim, cudaStream_t stream) {
+// x [rows <= 16, k_dim], w [n_out, k_dim], out [rows, n_out]; bf16; k_dim a multiple of 32.  act: -1 none, else the
+// activation of se_activation applied to the rounded product.
+extern "C" int se_gemv(const void* x, const void* w, void* out, int rows, int n_out, int k_dim, int act, cudaStream_t stream) {
     if (rows <= 0) return 0;
+    if (act < -1 || act > 3) return SE_ERR_ARGUMENT;
     if (!se_gemv_supported(rows, n_out, k_dim)) return SE_ERR_UNSUPPORTED;
     // Shape = 100 * (warps that split K) + (weight rows per block).  A warp's walk over its
     // share of K is one chain of dependent loads, so a long K takes more warps (measured:
@@ -133,8 +137,8 @@ extern "C" int se_gemv(const void* x, const void* w, void* out, int rows, int n_
     const int nt = rows <= 8 ? 1 : 2;
 #define SE_GEMV_CASE(W, R)                                                       \
     case W * 100 + R:                                                            \
-        if (nt == 1) launch_gemv<1, W, R>(x, w, out, rows, n_out, k_dim, stream); \
-        else launch_gemv<2, W, R>(x, w, out, rows, n_out, k_dim, stream);         \
+        if (nt == 1) launch_gemv<1, W, R>(x, w, out, rows, n_out, k_dim, act, stream); \
+        else launch_gemv<2, W, R>(x, w, out, rows, n_out, k_dim, act, stream);         \
         break;
     switch (shape) {
         SE_GEMV_CASE(4, 8) SE_GEMV_CASE(4, 16) SE_GEMV_CASE(8, 8) SE_GEMV_CASE(8, 16) SE_GEMV_CASE(16, 8) SE_GEMV_CASE(16, 16)

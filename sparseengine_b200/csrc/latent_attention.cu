@@ -37,40 +37,102 @@ __device__ __forceinline__ float rotated_element(const T* x, int i, int pos, con
     return first ? u * cs - w * sn : w * cs + u * sn;
 }
 
+// The rotated parts of a token's query heads into the query rows of the tiled kernel, qfull[t, h, rank + i]; all
+// threads of the block, cos and sin of the token's angles in shared memory.
+template <typename T>
+__device__ __forceinline__ void rotate_queries(const T* q_row, int d, T* dst, int heads, int rank, int rot, int rotary_dim,
+                                               int interleaved, const float* cs_t, const float* sn_t) {
+    const int half = rotary_dim / 2, D = rank + rot;
+    // 8 dims (neighbouring pairs) or 8 and 8 (split halves) at a time where sizes and addresses allow it
+    if (rotary_dim == rot && rot > 0 && ((interleaved ? rot : half) & 7) == 0 && (d & 7) == 0 && (rank & 7) == 0 && aligned8(q_row) &&
+        aligned8(dst)) {
+        const int items = (interleaved ? rot : half) / 8;
+        for (int x = threadIdx.x; x < heads * items; x += blockDim.x) {
+            const int h = x / items, i = (x - h * items) * 8;
+            const T* src = q_row + (size_t)h * (d + rot) + d;
+            T* out = dst + (size_t)h * D + rank;
+            float u[8], w[8], o[8];
+            load8(src + i, u);
+            if (interleaved) {
+#pragma unroll
+                for (int j = 0; j < 8; j += 2) {
+                    const float cs = cs_t[(i + j) / 2], sn = sn_t[(i + j) / 2];
+                    o[j] = u[j] * cs - u[j + 1] * sn;
+                    o[j + 1] = u[j + 1] * cs + u[j] * sn;
+                }
+                store8(out + i, o);
+            } else {
+                load8(src + half + i, w);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    o[j] = u[j] * cs_t[i + j] - w[j] * sn_t[i + j];
+                    w[j] = w[j] * cs_t[i + j] + u[j] * sn_t[i + j];
+                }
+                store8(out + i, o);
+                store8(out + half + i, w);
+            }
+        }
+        return;
+    }
+    const int items = half + rot - rotary_dim;           // per head: pairs, then single dims that pass
+    for (int x = threadIdx.x; x < heads * items; x += blockDim.x) {
+        const int h = x / items, k = x - h * items;
+        const T* src = q_row + (size_t)h * (d + rot) + d;
+        T* out = dst + (size_t)h * D + rank;
+        if (k >= half) { out[rotary_dim + k - half] = src[rotary_dim + k - half]; continue; }
+        const int a = interleaved ? 2 * k : k, b = interleaved ? 2 * k + 1 : k + half;
+        const float u = to_float(src[a]), w = to_float(src[b]), cs = cs_t[k], sn = sn_t[k];
+        out[a] = from_float<T>(u * cs - w * sn);
+        out[b] = from_float<T>(w * cs + u * sn);
+    }
+}
+
 // One block per token.  proj row: [q latent (q_rank) | kv latent (rank) | shared key part (rot)].
 //   cq_out[t]           = rmsnorm(q latent) * q_w                      (activation type; q_rank 0: queries have no latent)
 //   page row [0, rank)  = rmsnorm(kv latent) * kv_w
 //   page row [rank, ..) = the key part, rotated by the position (rotated_element)
+// With q (rows q_pitch apart, [heads * (d + rot)]; nullptr: none) also the rotated parts of the queries into qfull
+// [tokens, heads, rank + rot].
 template <typename T>
 __global__ void latent_prep_kernel(const T* proj, int proj_stride, const T* __restrict__ q_w, const T* __restrict__ kv_w,
                                    const float* __restrict__ inv_freq, const int* __restrict__ positions,
                                    const int* __restrict__ token_seq, const int* __restrict__ seq_rows,
                                    const int* __restrict__ table, int table_stride, T* cache, T* cq_out, int q_rank,
                                    int rank, int rot, int rotary_dim, int interleaved, float eps, int page_size,
-                                   int num_pages, int write_cache, int* error) {
+                                   int num_pages, int write_cache, const T* q, int q_pitch, int heads, int d, T* qfull,
+                                   int* error) {
+    extern __shared__ float cs_sn[];             // [rotary_dim / 2] cos, then as many sin
     __shared__ float scratch[33];
+    grid_dependency_trigger();
     const int t = blockIdx.x;
+    const int half = rotary_dim / 2;
+    float* cs_t = cs_sn;
+    float* sn_t = cs_sn + half;
+    grid_dependency_wait();                      // the step's inputs are older, but were maybe copied just before the kernel ahead
+    const int pos = positions[t];
+    for (int k = threadIdx.x; k < half; k += blockDim.x) sincosf((float)pos * inv_freq[k], &sn_t[k], &cs_t[k]);
     const T* row = proj + (size_t)t * proj_stride;
-    float sq = 0.f, sk = 0.f;
+    float sk = 0.f;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_float(row[q_rank + i]); sk += v * v; }
-    const float inv_k = 1.0f / sqrtf(block_sum(sk, scratch) / (float)rank + eps);
+    const float inv_k = 1.0f / sqrtf(block_sum(sk, scratch) / (float)rank + eps);       // its barriers also publish the angles
     if (q_rank > 0) {
+        float sq = 0.f;
         for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = to_float(row[i]); sq += v * v; }
         const float inv_q = 1.0f / sqrtf(block_sum(sq, scratch) / (float)q_rank + eps);
         for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
             cq_out[(size_t)t * q_rank + i] = from_float<T>(to_float(row[i]) * inv_q * to_float(q_w[i]));
     }
+    if (q != nullptr)
+        rotate_queries(q + (size_t)t * q_pitch, d, qfull + (size_t)t * heads * (rank + rot), heads, rank, rot, rotary_dim, interleaved,
+                       cs_t, sn_t);
     if (!write_cache) return;
-    const int pos = positions[t];
     const int page = table[(size_t)seq_rows[token_seq[t]] * table_stride + pos / page_size];
     if (!page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_LATENT_PREP)) return;
     const int D = rank + rot;
     T* dst = cache + ((size_t)page * page_size + pos % page_size) * D;
     for (int i = threadIdx.x; i < rank; i += blockDim.x)
         dst[i] = from_float<T>(to_float(row[q_rank + i]) * inv_k * to_float(kv_w[i]));
-    const T* kr = row + q_rank + rank;
-    for (int i = threadIdx.x; i < rot; i += blockDim.x)
-        dst[rank + i] = from_float<T>(rotated_element(kr, i, pos, inv_freq, rotary_dim, interleaved));
+    rotate_queries(row + q_rank + rank, 0, dst, 1, rank, rot, rotary_dim, interleaved, cs_t, sn_t);     // one "head"
 }
 
 constexpr int kLatWarps = 4;
@@ -158,18 +220,27 @@ __global__ void latent_attention_plain_kernel(const float* __restrict__ q_lat, c
 
 extern "C" int se_latent_max_row() { return 32 * 32; }
 
+// q (nullptr: none), q_pitch, heads, d, qfull: the rotated parts of the queries into the tiled kernel's query rows.
 extern "C" int se_latent_prep(const void* proj, int proj_stride, const void* q_w, const void* kv_w, const float* inv_freq,
                               const int* positions, const int* token_seq, const int* seq_rows, const int* table,
                               int table_stride, void* cache, void* cq_out, int tokens, int q_rank, int rank, int rot,
                               int rotary_dim, int interleaved, float eps, int page_size, int num_pages, int write_cache,
-                              int* error, int dtype, cudaStream_t stream) {
+                              const void* q, int q_pitch, int heads, int d, void* qfull, int* error, int dtype,
+                              cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (q_rank < 0 || (q_rank > 0 && (q_w == nullptr || cq_out == nullptr)) || rank <= 0 || rot < 0 || rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || page_size <= 0)
+    if (q_rank < 0 || (q_rank > 0 && (q_w == nullptr || cq_out == nullptr)) || rank <= 0 || rot < 0 || rotary_dim < 0 ||
+        rotary_dim > rot || (rotary_dim & 1) || page_size <= 0)
         return SE_ERR_ARGUMENT;
-    SE_DISPATCH_DTYPE(dtype, T,
-        se::latent_prep_kernel<T><<<tokens, 128, 0, stream>>>((const T*)proj, proj_stride, (const T*)q_w, (const T*)kv_w,
-            inv_freq, positions, token_seq, seq_rows, table, table_stride, (T*)cache, (T*)cq_out, q_rank, rank, rot,
-            rotary_dim, interleaved, eps, page_size, num_pages, write_cache, error));
+    if (q != nullptr && (qfull == nullptr || heads <= 0 || d < 0 || q_pitch < heads * (d + rot))) return SE_ERR_ARGUMENT;
+    if (rank + rot > se_latent_max_row()) return SE_ERR_UNSUPPORTED;
+    const int threads = q != nullptr && heads * rot >= 1024 ? 256 : 128;
+    SE_DISPATCH_DTYPE(dtype, T, {
+        cudaError_t e = SE_LAUNCH_DEPENDENT("lat", se::latent_prep_kernel<T>, dim3(tokens), dim3(threads),
+            (size_t)rotary_dim * sizeof(float), stream, (const T*)proj, proj_stride, (const T*)q_w, (const T*)kv_w, inv_freq,
+            positions, token_seq, seq_rows, table, table_stride, (T*)cache, (T*)cq_out, q_rank, rank, rot, rotary_dim,
+            interleaved, eps, page_size, num_pages, write_cache, (const T*)q, q_pitch, heads, d, (T*)qfull, error);
+        if (e != cudaSuccess) return (int)e;
+    });
     SE_LAUNCH_CHECK();
 }
 
@@ -224,20 +295,20 @@ constexpr int kThreads = 32 * kWarps;
 
 using namespace se::mma;
 
-// qfull[t, h, :] = [q_lat[h, t, :] | rotated part of q[t, h]] in bfloat16: the query rows as the tiled kernel reads them
-__global__ void latent_q_pack_kernel(const float* __restrict__ q_lat, const __nv_bfloat16* __restrict__ q, int q_pitch,
-                                     int d, const float* __restrict__ inv_freq, int rotary_dim, int interleaved,
-                                     const int* __restrict__ positions, __nv_bfloat16* __restrict__ qfull, int tokens,
-                                     int heads, int rank, int rot) {
-    const int t = blockIdx.x, h = blockIdx.y;
-    const int D = rank + rot;
-    __nv_bfloat16* dst = qfull + ((size_t)t * heads + h) * D;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x)
-        dst[i] = __float2bfloat16_rn(q_lat[((size_t)h * tokens + t) * rank + i]);
-    const __nv_bfloat16* qr = q + (size_t)t * q_pitch + (size_t)h * (d + rot) + d;
-    const int pos = positions[t];
-    for (int i = threadIdx.x; i < rot; i += blockDim.x)
-        dst[rank + i] = __float2bfloat16_rn(rotated_element(qr, i, pos, inv_freq, rotary_dim, interleaved));
+// qfull[t, h, rank ..] = rotated part of q[t, h]: the query rows as the tiled kernel reads them (their first `rank` dims are
+// the queries in the latent's space, which a matrix product outside this file writes).  One block per token.
+__global__ void latent_q_rotate_kernel(const __nv_bfloat16* q, int q_pitch, int d, const float* __restrict__ inv_freq,
+                                       int rotary_dim, int interleaved, const int* __restrict__ positions,
+                                       __nv_bfloat16* qfull, int heads, int rank, int rot) {
+    extern __shared__ float cs_sn[];
+    grid_dependency_trigger();
+    grid_dependency_wait();
+    const int t = blockIdx.x, half = rotary_dim / 2;
+    for (int k = threadIdx.x; k < half; k += blockDim.x)
+        sincosf((float)positions[t] * inv_freq[k], &cs_sn[half + k], &cs_sn[k]);
+    __syncthreads();
+    rotate_queries(q + (size_t)t * q_pitch, d, qfull + (size_t)t * heads * (rank + rot), heads, rank, rot, rotary_dim, interleaved,
+                   cs_sn, cs_sn + half);
 }
 
 // D16T, RT: the row's 16-dim groups rounded up to a multiple of four (the tile's chunks between the row's end and that
@@ -472,27 +543,42 @@ latent_attention_tiled_kernel(const __nv_bfloat16* __restrict__ qfull, const __n
     }
 }
 
-// One block per (token, head): the splits' sums brought to one maximum, the sink added once.
+// One block per (token, head): the splits' sums brought to one maximum, the sink added once.  The splits' factors are
+// computed once by the block's first warp; then every thread sums its columns over the splits.
 __global__ void latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                               const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int tokens,
                                               int heads, int rank, int splits, float scale) {
+    extern __shared__ float factor[];            // [splits], already divided by the sum
     const int t = blockIdx.x, h = blockIdx.y;
     const size_t at = ((size_t)t * heads + h) * splits;
     const float scale_log2 = scale * 1.4426950408889634f;
-    float mt = sink != nullptr ? sink[h] / scale : -INFINITY;
-    for (int z = 0; z < splits; ++z) mt = fmaxf(mt, part_ml[2 * (at + z)]);
-    float lt = sink != nullptr ? exp2f((sink[h] / scale - mt) * scale_log2) : 0.f;
-    for (int z = 0; z < splits; ++z) {
-        const float m = part_ml[2 * (at + z)];
-        if (m != -INFINITY) lt += part_ml[2 * (at + z) + 1] * exp2f((m - mt) * scale_log2);
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x;
+        const float sk = sink != nullptr ? sink[h] / scale : -INFINITY;
+        float mt = sk;
+        for (int z = lane; z < splits; z += 32) mt = fmaxf(mt, part_ml[2 * (at + z)]);
+        mt = warp_max(mt);
+        float lt = 0.f;
+        for (int z = lane; z < splits; z += 32) {
+            const float m = part_ml[2 * (at + z)];
+            const float f = m == -INFINITY ? 0.f : exp2f((m - mt) * scale_log2);
+            factor[z] = f;
+            lt += f > 0.f ? part_ml[2 * (at + z) + 1] * f : 0.f;
+        }
+        lt = warp_sum(lt);
+        if (sink != nullptr) lt += exp2f((sk - mt) * scale_log2);
+        for (int z = lane; z < splits; z += 32) factor[z] /= lt;
     }
+    __syncthreads();
     for (int c = threadIdx.x; c < rank; c += blockDim.x) {
         float o = 0.f;
+#pragma unroll 8
         for (int z = 0; z < splits; ++z) {
-            const float m = part_ml[2 * (at + z)];
-            if (m != -INFINITY) o += part_o[(at + z) * rank + c] * exp2f((m - mt) * scale_log2);
+            const float f = factor[z];
+            const float v = part_o[(at + z) * rank + c];
+            o += f > 0.f ? v * f : 0.f;          // a split without keys holds zeros
         }
-        out[((size_t)t * heads + h) * rank + c] = __float2bfloat16_rn(o / lt);
+        out[((size_t)t * heads + h) * rank + c] = __float2bfloat16_rn(o);
     }
 }
 
@@ -517,7 +603,7 @@ static int launch_tiled(const void* qfull, const void* cache, const int* table, 
         (__nv_bfloat16*)out, tokens, heads, rank, rot, page_size, scale, window, num_pages, error, splits, tiles_per_split,
         part_o, part_ml);
     if (splits > 1)
-        latent_attention_merge_kernel<<<dim3(tokens, heads), 64, 0, stream>>>(part_o, part_ml, sink, (__nv_bfloat16*)out,
+        latent_attention_merge_kernel<<<dim3(tokens, heads), rank > 64 ? 128 : 64, splits * sizeof(float), stream>>>(part_o, part_ml, sink, (__nv_bfloat16*)out,
                                                                              tokens, heads, rank, splits, scale);
     return (int)cudaGetLastError();
 }
@@ -530,14 +616,18 @@ extern "C" int se_latent_attention_tiled_supported(int rank, int rot) {
     return rank > 0 && rot >= 0 && rank % 16 == 0 && rot % 16 == 0 && rank + rot <= 256;
 }
 
-extern "C" int se_latent_q_pack(const float* q_lat, const void* q, int q_pitch, int d, const float* inv_freq,
-                                int rotary_dim, int interleaved, const int* positions, void* qfull, int tokens, int heads, int rank, int rot,
-                                cudaStream_t stream) {
+extern "C" int se_latent_q_rotate(const void* q, int q_pitch, int d, const float* inv_freq, int rotary_dim, int interleaved,
+                                  const int* positions, void* qfull, int tokens, int heads, int rank, int rot,
+                                  cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (heads <= 0 || heads > 65535 || rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || q_pitch < heads * (d + rot))
+    if (heads <= 0 || rank <= 0 || rot < 0 || rotary_dim < 0 || rotary_dim > rot || (rotary_dim & 1) || d < 0 ||
+        q_pitch < heads * (d + rot))
         return SE_ERR_ARGUMENT;
-    se::lat::latent_q_pack_kernel<<<dim3(tokens, heads), 64, 0, stream>>>(
-        q_lat, (const __nv_bfloat16*)q, q_pitch, d, inv_freq, rotary_dim, interleaved, positions, (__nv_bfloat16*)qfull, tokens, heads, rank, rot);
+    if (rank + rot > se_latent_max_row()) return SE_ERR_UNSUPPORTED;
+    cudaError_t e = SE_LAUNCH_DEPENDENT("lat", se::lat::latent_q_rotate_kernel, dim3(tokens), dim3(256),
+        (size_t)rotary_dim * sizeof(float), stream, (const __nv_bfloat16*)q, q_pitch, d, inv_freq, rotary_dim, interleaved,
+        positions, (__nv_bfloat16*)qfull, heads, rank, rot);
+    if (e != cudaSuccess) return (int)e;
     SE_LAUNCH_CHECK();
 }
 
@@ -554,7 +644,7 @@ extern "C" int se_latent_attention_tiled(const void* qfull, const void* cache, c
                                          cudaStream_t stream) {
     if (entries <= 0 || max_q_len <= 0) return 0;
     if (!se_latent_attention_tiled_supported(rank, rot) || heads <= 0 || heads > 65535) return SE_ERR_UNSUPPORTED;
-    if (!(scale > 0.f) || page_size <= 0 || splits < 1 || splits > 65535) return SE_ERR_ARGUMENT;
+    if (!(scale > 0.f) || page_size <= 0 || splits < 1 || splits > 8192) return SE_ERR_ARGUMENT;
     if (splits > 1 && (tiles_per_split < 1 || part_o == nullptr || part_ml == nullptr)) return SE_ERR_ARGUMENT;
     if (tile_keys != 64 && tile_keys != 32) return SE_ERR_ARGUMENT;
     const int d16t = (rank + rot + 63) / 64 * 4, rt = (rank + 63) / 64 * 4;

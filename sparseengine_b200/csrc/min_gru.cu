@@ -28,9 +28,14 @@ constexpr int kTile = kWarps * kTokens;      // tokens of a CTA at a time
 constexpr int kChannels = 64;                // channels of a CTA: two per lane
 constexpr int kMaxCluster = 8;
 
-// 16-bit activations take the fast exponential and division (a few units in the last place of 32-bit)
+// 16-bit activations take the special-function unit's exponential and reciprocal (a few units in the last place of
+// 32-bit; beyond their range the results are 0 and 1, as they should be)
 template <typename T> __device__ __forceinline__ float sigmoid(float x) {
-    return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-x)) : 1.f / (1.f + expf(-x));
+    if (sizeof(T) != 2) return 1.f / (1.f + expf(-x));
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+    return r;
 }
 template <typename T> __device__ __forceinline__ void cell(float zl, float u, float& keep, float& add) {
     const float z = sigmoid<T>(zl);
@@ -57,6 +62,17 @@ template <bool PAIR, typename T> __device__ __forceinline__ void write2(T* row, 
     row[c] = from_float<T>(v.x);
     if (c + 1 < width) row[c + 1] = from_float<T>(v.y);
 }
+
+// the same as stored (a register for a pair of bfloat16), to be unpacked later
+template <typename T> struct Stored { using type = float2; };
+template <> struct Stored<__nv_bfloat16> { using type = __nv_bfloat162; };
+template <bool PAIR> __device__ __forceinline__ float2 read_stored(const float* row, int c, int width) { return read2<PAIR>(row, c, width); }
+template <bool PAIR> __device__ __forceinline__ __nv_bfloat162 read_stored(const __nv_bfloat16* row, int c, int width) {
+    if (PAIR) return *reinterpret_cast<const __nv_bfloat162*>(row + c);
+    return __halves2bfloat162(row[c], c + 1 < width ? row[c + 1] : row[c]);
+}
+__device__ __forceinline__ float2 unpack(float2 v) { return v; }
+__device__ __forceinline__ float2 unpack(__nv_bfloat162 v) { return __bfloat1622float2(v); }
 
 template <typename T, bool PAIR>
 __global__ void __launch_bounds__(128)
@@ -113,31 +129,34 @@ min_gru_chunk_kernel(const T* __restrict__ proj, int pitch, const float* __restr
         const int t0 = base + rank * kTile + warp * kTokens;
         const int n = min(max(q_len - t0, 0), kTokens);
         const T* row = proj + (size_t)(tok0 + t0) * pitch;
-        float2 keep[kTokens], add[kTokens], g[kTokens];
-#pragma unroll
-        for (int i = 0; i < kTokens; ++i) {
-            keep[i] = add[i] = g[i] = make_float2(0.f, 0.f);
-            if (i < n) {
-                keep[i] = read2<PAIR>(row + (size_t)i * pitch, cc, width);
-                add[i] = read2<PAIR>(row + (size_t)i * pitch + width, cc, width);
-            }
-        }
+        float2 keep[kTokens], add[kTokens];
+        typename Stored<T>::type gates[kTokens];
         float2 A = make_float2(1.f, 1.f), B = make_float2(0.f, 0.f);
+        if (n > 0) {
+            // No branch between the tokens (their chains of special functions overlap): a token beyond the last is
+            // the last one read again, and changes nothing.
 #pragma unroll
-        for (int i = 0; i < kTokens; ++i) {
-            if (i < n) {
+            for (int i = 0; i < kTokens; ++i) {
+                const T* r = row + (size_t)min(i, n - 1) * pitch;
+                keep[i] = read2<PAIR>(r, cc, width);
+                add[i] = read2<PAIR>(r + width, cc, width);
+                gates[i] = read_stored<PAIR>(r + 2 * width, cc, width);
+            }
+#pragma unroll
+            for (int i = 0; i < kTokens; ++i) {
                 const float2 z = keep[i], u = add[i];
                 cell<T>(z.x + bz.x, u.x + bu.x, keep[i].x, add[i].x);
                 cell<T>(z.y + bz.y, u.y + bu.y, keep[i].y, add[i].y);
+                if (i >= n) { keep[i] = make_float2(1.f, 1.f); add[i] = make_float2(0.f, 0.f); }
+            }
+#pragma unroll
+            for (int i = 0; i < kTokens; ++i) {
                 A.x *= keep[i].x; B.x = keep[i].x * B.x + add[i].x;
                 A.y *= keep[i].y; B.y = keep[i].y * B.y + add[i].y;
             }
         }
         warp_ab[buf][warp][2 * lane] = make_float2(A.x, B.x);
         warp_ab[buf][warp][2 * lane + 1] = make_float2(A.y, B.y);
-#pragma unroll
-        for (int i = 0; i < kTokens; ++i)                        // asked for here, used after the exchange
-            if (i < n) g[i] = read2<PAIR>(row + (size_t)i * pitch + 2 * width, cc, width);
         __syncthreads();
         if (threadIdx.x < kChannels) {
             float2 f = warp_ab[buf][0][threadIdx.x];
@@ -167,13 +186,16 @@ min_gru_chunk_kernel(const T* __restrict__ proj, int pitch, const float* __restr
             s.x = a.x * s.x + a.y;
             s.y = b.x * s.y + b.y;
         }
-        T* dst = out + (size_t)(tok0 + t0) * width;
+        if (n > 0) {
+            T* dst = out + (size_t)(tok0 + t0) * width;
+            const int last = live ? n : 0;
 #pragma unroll
-        for (int i = 0; i < kTokens; ++i) {
-            if (i < n) {
+            for (int i = 0; i < kTokens; ++i) {
                 s.x = keep[i].x * s.x + add[i].x;
                 s.y = keep[i].y * s.y + add[i].y;
-                if (live) write2<PAIR>(dst + (size_t)i * width, cc, width, make_float2(s.x * silu<T>(g[i].x), s.y * silu<T>(g[i].y)));
+                const float2 g = unpack(gates[i]);
+                const float2 y = make_float2(s.x * silu<T>(g.x), s.y * silu<T>(g.y));
+                if (i < last) write2<PAIR>(dst + (size_t)i * width, cc, width, y);
             }
         }
     }

@@ -381,22 +381,24 @@ def _interleaved(pairing: str) -> int:
 
 
 def latent_prep(proj, q_w, kv_w, inv_freq, positions, token_seq, seq_rows, table, cache, cq_out, *, q_rank, rank, rot,
-                rotary_dim, eps, page_size, write_cache=True, num_pages=None, pairing: str = "split_half"):
+                rotary_dim, eps, page_size, write_cache=True, num_pages=None, pairing: str = "split_half", queries=None):
     """From a step's rows ``[q latent | kv latent | shared key part]``: the normalised query latent
     (``cq_out``; ``q_rank`` 0: there is none), and into each token's page slot the normalised kv latent and
-    the rotated key part."""
+    the rotated key part.  ``queries = (q, heads, head_dim, qfull)``: also :func:`latent_q_rotate`."""
     tokens = proj.shape[0]
     dt = proj.dtype
     if proj.dim() != 2 or proj.stride(1) != 1 or proj.shape[1] != q_rank + rank + rot:
         raise ValueError("proj must be [tokens, q_rank + rank + rot] with contiguous rows")
-    _check(_fn("se_latent_prep", "pippp" "ppp" "pi" "pp" "iiiiii" "f" "iii" "p" "ip")(
+    _check(_fn("se_latent_prep", "pippp" "ppp" "pi" "pp" "iiiiii" "f" "iii" "piiip" "p" "ip")(
         proj.data_ptr(), proj.stride(0), _ptr(q_w, dt, "q_norm"), _ptr(kv_w, dt, "kv_norm"),
         _ptr(inv_freq, torch.float32, "inv_freq"), _ptr(positions, torch.int32, "positions"),
         _ptr(token_seq, torch.int32, "token_seq"), _ptr(seq_rows, torch.int32, "seq_rows"),
         _ptr(table, torch.int32, "table"), table.shape[1], _ptr(cache, dt, "cache"), _ptr(cq_out, dt, "cq_out"),
         tokens, q_rank, rank, rot, rotary_dim, _interleaved(pairing), float(eps), page_size,
-        cache.shape[0] if num_pages is None else int(num_pages), int(bool(write_cache)), _ptr(error_word(proj.device)),
-        dtype_code(dt), _stream()), "latent_prep")
+        cache.shape[0] if num_pages is None else int(num_pages), int(bool(write_cache)),
+        *((_rows_ptr(queries[0], "q", dt), queries[0].stride(0), queries[1], queries[2], _ptr(queries[3], dt, "qfull"))
+          if queries is not None else (None, 0, 0, 0, None)),
+        _ptr(error_word(proj.device)), dtype_code(dt), _stream()), "latent_prep")
     return cq_out
 
 
@@ -425,15 +427,14 @@ def latent_attention_tiled_supported(rank: int, rot: int) -> bool:
     return rank > 0 and rot >= 0 and rank % 16 == 0 and rot % 16 == 0 and rank + rot <= 256
 
 
-def latent_q_pack(q_lat, q, inv_freq, positions, qfull, *, heads, head_dim, rank, rot, rotary_dim,
-                  pairing: str = "split_half"):
-    """``qfull[t, h] = [q_lat[h, t] | rotated part of q[t, h]]`` in bfloat16: the query rows of the tiled kernel.
-    ``q``'s rows may be a view with a pitch."""
+def latent_q_rotate(q, inv_freq, positions, qfull, *, heads, head_dim, rank, rot, rotary_dim, pairing: str = "split_half"):
+    """``qfull[t, h, rank:] = rotated part of q[t, h]`` (bfloat16): the query rows of the tiled kernel, whose first
+    ``rank`` dims a matrix product writes.  ``q``'s rows may be a view with a pitch."""
     tokens = q.shape[0]
-    _check(_fn("se_latent_q_pack", "ppiipii" "pp" "iiii" "p")(
-        _ptr(q_lat, torch.float32, "q_lat"), _rows_ptr(q, "q", torch.bfloat16), q.stride(0), head_dim,
-        _ptr(inv_freq, torch.float32, "inv_freq"), rotary_dim, _interleaved(pairing), _ptr(positions, torch.int32, "positions"), _ptr(qfull, torch.bfloat16, "qfull"), tokens, heads, rank,
-        rot, _stream()), "latent_q_pack")
+    _check(_fn("se_latent_q_rotate", "piipii" "pp" "iiii" "p")(
+        _rows_ptr(q, "q", torch.bfloat16), q.stride(0), head_dim, _ptr(inv_freq, torch.float32, "inv_freq"), rotary_dim,
+        _interleaved(pairing), _ptr(positions, torch.int32, "positions"), _ptr(qfull, torch.bfloat16, "qfull"), tokens, heads,
+        rank, rot, _stream()), "latent_q_rotate")
     return qfull
 
 
@@ -711,14 +712,25 @@ def min_gru_scan(proj, bias, state, step, out):
     return out
 
 
+def min_gru_plan(entries: int, width: int, max_q_len: int, sms: Optional[int] = None) -> int:
+    """CTAs per cluster of the chunked minGRU (64 channels and 128 tokens at a time each): 1, 2, 4 or 8, no more than
+    the longest entry fills, and no more than give the device 1.5 CTAs per SM (two fit; an exchange between fewer CTAs is
+    cheaper).  Measured, one 2,048-token prompt: 2,048 channels 15.8 us with 8, 18.6 with 4; 4,096 channels 27.0 with 4, 28.4
+    with 8; four such prompts of 4,096 channels 102 with 1, 117 with 8."""
+    if sms is None:
+        sms = sm_count()
+    blocks, ctas = entries * -(-width // 64), 1
+    while ctas < 8 and ctas * 128 < max_q_len and 2 * ctas * blocks < 3 * sms:
+        ctas *= 2
+    return ctas
+
+
 def min_gru_chunk(proj, bias, state, step, out, ctas=None):
-    """:func:`min_gru_scan` with a request's tokens dealt out to the warps of a cluster of ``ctas`` CTAs (128 tokens each
-    at a time; default: as many as the longest entry fills, at most 8): for steps with prompt portions."""
+    """:func:`min_gru_scan` with a request's tokens dealt out to the warps of a cluster of ``ctas`` CTAs (default:
+    :func:`min_gru_plan`): for steps with prompt portions."""
     width = out.shape[1]
     if ctas is None:
-        ctas = 1
-        while ctas < 8 and ctas * 128 < step.max_q_len:
-            ctas *= 2
+        ctas = min_gru_plan(step.num_seqs, width, step.max_q_len, sm_count(proj.device))
     _check(_fn("se_min_gru_chunk", "pip" "pl" "ppp" "iiii" "p")(
         _rows_ptr(proj, "proj"), proj.stride(0), _ptr(bias, torch.float32, "bias"), _ptr(state, torch.float32, "state"),
         state.stride(0), _ptr(step.cu_q), _ptr(step.seq_rows), _ptr(out, proj.dtype, "out"), step.num_seqs, width, int(ctas),
@@ -1171,13 +1183,14 @@ def gemv_supported(rows: int, n_out: int, k_dim: int) -> bool:
     return 1 <= rows <= 16 and n_out >= 1 and k_dim >= 32 and k_dim % 32 == 0
 
 
-def gemv(x, w, out):
-    """out[rows <= 16, n] = x · wᵀ, weights streamed once through tensor-core fragments."""
+def gemv(x, w, out, activation=None):
+    """out[rows <= 16, n] = x · wᵀ, weights streamed once through tensor-core fragments.  ``activation``: a name of
+    :data:`ACTIVATIONS` applied to the rounded product."""
     rows, k_dim = x.shape
     n_out = w.shape[0]
-    _check(_fn("se_gemv", "pppiiip")(
+    _check(_fn("se_gemv", "pppiiiip")(
         _ptr(x, torch.bfloat16, "x"), _ptr(w, torch.bfloat16, "w"), _ptr(out, torch.bfloat16, "out"), rows, n_out,
-        k_dim, _stream()), "gemv")
+        k_dim, -1 if activation is None else ACTIVATIONS[activation], _stream()), "gemv")
     return out
 
 

@@ -217,6 +217,58 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
     }
 }
 
+// Per-head norms (per_head 1 with weights, 2 without) and nothing else: no rotation, temperature, bias or blending.
+// Every 16-byte chunk (float32: two) of the step's projection rows is a lane's work item; a head's LANES = d / 8
+// chunks lie in neighbouring lanes of one warp, so its sum of squares is a few shuffles and each input is read once.
+template <typename T, int LANES>
+__global__ void __launch_bounds__(256)
+qk_prep_heads_kernel(const T* proj, int pitch, const T* __restrict__ q_w, const T* __restrict__ k_w,
+                     const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ seq_rows,
+                     const int* __restrict__ table, int table_stride, T* cache, T* q_out, long long items, int hq, int hkv,
+                     int dv, float eps, int page_size, int num_pages, int* __restrict__ error) {
+    constexpr int d = 8 * LANES;
+    grid_dependency_trigger();
+    grid_dependency_wait();
+    const int qc = hq * LANES, kc = hkv * LANES, per_token = qc + kc + hkv * (dv / 8);
+    const long long x = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    const bool live = x < items;
+    const int t = live ? (int)(x / per_token) : 0;
+    const int c = live ? (int)(x - (long long)t * per_token) : 0;
+    float v[8];
+    load8(proj + (size_t)t * pitch + 8 * c, v);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);       // items of values: a sum nobody uses
+    if (!live) return;
+    const int in_head = (c % LANES) * 8;
+    if (c < qc + kc) {
+        const T* w = c < qc ? q_w : k_w;
+        const float inv = 1.0f / sqrtf(ss / (float)d + eps);
+        float wv[8];
+        if (w != nullptr) load8(w + in_head, wv);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] *= w != nullptr ? inv * wv[j] : inv;
+    }
+    if (c < qc) {
+        store8(q_out + ((size_t)t * qc + c) * 8, v);
+        return;
+    }
+    const int pos = positions[t];
+    const int page = table[(size_t)seq_rows[token_seq[t]] * table_stride + pos / page_size];
+    if (!page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_QK_PREP)) return;
+    const int slot = pos % page_size;
+    T* base = cache + (size_t)page * hkv * page_size * (d + dv);
+    if (c < qc + kc) {
+        const int h = (c - qc) / LANES;
+        store8(base + ((size_t)h * page_size + slot) * d + in_head, v);
+    } else {
+        const int i = (c - qc - kc) * 8, h = i / dv;
+        store8(base + (size_t)hkv * page_size * d + ((size_t)h * page_size + slot) * dv + (i - h * dv), v);
+    }
+}
+
 }  // namespace se
 
 extern "C" int se_qk_prep_general(const void* proj, int pitch, const void* q_w, const void* k_w, const float* inv_freq,
@@ -232,6 +284,28 @@ extern "C" int se_qk_prep_general(const void* proj, int pitch, const void* q_w, 
     if (rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) || (rotary_dim > 0 && inv_freq == nullptr)) return SE_ERR_ARGUMENT;
     if (rotary_dim > 2 * se::kMaxHalf) return SE_ERR_UNSUPPORTED;
     if (v_first != nullptr && (v_mix == nullptr || !has_kv || v_first_pitch < hkv * dv)) return SE_ERR_ARGUMENT;
+    // heads of 64, 128 or 256 elements that are normed and nothing else
+    const size_t esize = dtype == SE_DTYPE_F32 ? 4 : 2;
+    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int lanes = d / 8;
+    if (has_kv && per_head && rotary_dim == 0 && (temp_coef == 0.f || temp_every <= 0) && v_first == nullptr && bias == nullptr &&
+        (per_head == 2 || (q_w != nullptr && k_w != nullptr)) && (d == 64 || d == 128 || d == 256) && (dv & 7) == 0 &&
+        (hkv * (dv / 8)) % lanes == 0 && (pitch * esize) % 16 == 0 && aligned(proj) && aligned(q_out) && aligned(cache) &&
+        (q_w == nullptr || aligned(q_w)) && (k_w == nullptr || aligned(k_w))) {
+        const long long items = (long long)tokens * ((hq + hkv) * lanes + hkv * (dv / 8));
+        const long long blocks = (items + 255) / 256;
+        if (blocks > 0x7fffffffLL) return SE_ERR_UNSUPPORTED;
+        const bool weights = per_head == 1;
+        SE_DISPATCH_DTYPE(dtype, T, {
+            auto kernel = d == 64 ? se::qk_prep_heads_kernel<T, 8> : d == 128 ? se::qk_prep_heads_kernel<T, 16> : se::qk_prep_heads_kernel<T, 32>;
+            cudaError_t e = SE_LAUNCH_DEPENDENT("qk", kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, pitch,
+                                                 weights ? (const T*)q_w : nullptr, weights ? (const T*)k_w : nullptr, positions,
+                                                 token_seq, seq_rows, table, table_stride, (T*)cache, (T*)q_out, items, hq, hkv, dv,
+                                                 eps, page_size, num_pages, error);
+            if (e != cudaSuccess) return (int)e;
+        });
+        SE_LAUNCH_CHECK();
+    }
     const size_t smem = per_head ? (size_t)(hq + (has_kv ? hkv : 0)) * sizeof(float) : 0;
     if (smem > 40 * 1024) return SE_ERR_UNSUPPORTED;
     SE_DISPATCH_DTYPE(dtype, T, {

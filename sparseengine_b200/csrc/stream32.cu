@@ -253,13 +253,6 @@ __global__ void rmsnorm_add_stream_kernel(float* stream, const T* y, const T* __
     }
 }
 
-__device__ __forceinline__ float act_apply(float v, int kind) {
-    if (kind == 0) { const float r = fmaxf(v, 0.f); return r * r; }                       // squared relu
-    if (kind == 1) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));   // gelu (tanh form)
-    if (kind == 2) return v / (1.f + expf(-v));                                           // silu
-    return fmaxf(v, 0.f);                                                                 // relu
-}
-
 template <typename T>
 __global__ void activation_kernel(T* x, size_t n, int kind) {
     grid_dependency_wait();

@@ -88,18 +88,33 @@ class LatentAttention(Mixer):
         else:
             rope = RotaryArgs(None, 0)
         proj = linear(x, self.down if s.q_rank else self.in_proj)
+        tiled = self.takes_tiles(x.dtype)
+        qfull = torch.empty(tokens, H, rank + r, dtype=x.dtype, device=dev) if tiled else None
         cq = torch.empty(tokens, s.q_rank, dtype=x.dtype, device=dev) if s.q_rank else None
+        q = proj[:, :self.q_cols]                                            # [tokens, H * (d + r)]
         ops.latent_prep(proj[:, self.q_cols:self.g_off + s.q_rank], self.q_norm if s.q_rank else None, self.kv_norm,
                         rope.inv_freq, step.positions, step.token_seq, step.seq_rows, slot.table, slot.kv, cq,
                         q_rank=s.q_rank, rank=rank, rot=r, rotary_dim=rope.rotary_dim, eps=s.norm_eps,
-                        page_size=slot.page_size, write_cache=slot.write_cache, pairing=rope.pairing)
-        q = linear(cq, self.uq) if s.q_rank else proj[:, :self.q_cols]       # [tokens, H * (d + r)]
-        # the unrotated queries in the latent's space: [H, tokens, d] x [H, d, rank], 32-bit out
-        q_plain = q.unflatten(1, (H, d + r))[:, :, :d].transpose(0, 1)
-        q_lat = torch.bmm(q_plain, self.uk.view(H, d, rank), out_dtype=torch.float32) if x.dtype != torch.float32 \
-            else torch.bmm(q_plain, self.uk.view(H, d, rank))
+                        page_size=slot.page_size, write_cache=slot.write_cache, pairing=rope.pairing,
+                        queries=(q, H, d, qfull) if tiled and not s.q_rank else None)
+        if s.q_rank:
+            q = linear(cq, self.uq)
+            if tiled:
+                ops.latent_q_rotate(q, rope.inv_freq, step.positions, qfull, heads=H, head_dim=d, rank=rank, rot=r,
+                                    rotary_dim=rope.rotary_dim, pairing=rope.pairing)
+        # the unrotated queries in the latent's space: [H, tokens, d] x [H, d, rank], in the tiled kernel's query rows
+        # or 32-bit
+        q_plain, uk = q.unflatten(1, (H, d + r))[:, :, :d].transpose(0, 1), self.uk.view(H, d, rank)
         out_lat = torch.empty(tokens, H, rank, dtype=x.dtype, device=dev)
-        self.attend(q_lat, q, rope, out_lat, step, slot)
+        if tiled:
+            torch.bmm(q_plain, uk, out=qfull[:, :, :rank].transpose(0, 1))
+            self.attend_tiled(qfull, out_lat, step, slot)
+        else:
+            q_lat = torch.bmm(q_plain, uk) if x.dtype == torch.float32 else torch.bmm(q_plain, uk, out_dtype=torch.float32)
+            ops.latent_attention_plain(q_lat, q, rope.inv_freq, slot.kv, slot.table, step.seq_rows, step.token_seq,
+                                       step.positions, self.sink, out_lat, heads=H, head_dim=d, rank=rank, rot=r,
+                                       rotary_dim=rope.rotary_dim, page_size=slot.page_size, scale=s.scale, window=s.window,
+                                       pairing=rope.pairing)
         # the values' up-projection per head, read from and written to token-major rows through strided views
         heads_out = torch.empty(tokens, H, s.v_head_dim, dtype=x.dtype, device=dev)
         torch.bmm(out_lat.transpose(0, 1), self.uv.view(H, s.v_head_dim, rank).transpose(1, 2), out=heads_out.transpose(0, 1))
@@ -110,26 +125,20 @@ class LatentAttention(Mixer):
 
     use_tensor_cores = None      # False: always the kernel with one block per (token, head)
 
-    def attend(self, q_lat, q, rope, out_lat, step, slot):
+    def takes_tiles(self, dtype) -> bool:
         """bfloat16 steps of sizes the tiled kernel takes (latent and rotated part in multiples of 16, a
         cached row of at most 256) run on tensor-core tiles whose rows are (token, head) pairs, prompt
         portions and single tokens alike; everything else one block per (token, head)."""
         s = self.spec
-        if (self.use_tensor_cores is not False and q.dtype == torch.bfloat16 and s.scale > 0
-                and ops.latent_attention_tiled_supported(s.kv_rank, s.rot_dim)):
-            qfull = torch.empty(q.shape[0], s.num_heads, s.kv_rank + s.rot_dim, dtype=q.dtype, device=q.device)
-            ops.latent_q_pack(q_lat, q, rope.inv_freq, step.positions, qfull, heads=s.num_heads, head_dim=s.head_dim,
-                              rank=s.kv_rank, rot=s.rot_dim, rotary_dim=rope.rotary_dim, pairing=rope.pairing)
-            ops.latent_attention_tiled(qfull, slot.kv, slot.table, step.seq_rows, step.cu_q, step.kv_len, self.sink,
-                                       out_lat, entries=step.num_seqs, max_q_len=step.max_q_len, heads=s.num_heads,
-                                       rank=s.kv_rank, rot=s.rot_dim, page_size=slot.page_size, scale=s.scale,
-                                       window=s.window,
-                                       max_keys=step.max_kv_len if s.window is None else min(step.max_kv_len, s.window + step.max_q_len - 1))
-            return
-        ops.latent_attention_plain(q_lat, q, rope.inv_freq, slot.kv, slot.table, step.seq_rows, step.token_seq,
-                                   step.positions, self.sink, out_lat, heads=s.num_heads, head_dim=s.head_dim,
-                                   rank=s.kv_rank, rot=s.rot_dim, rotary_dim=rope.rotary_dim, page_size=slot.page_size,
-                                   scale=s.scale, window=s.window, pairing=rope.pairing)
+        return (self.use_tensor_cores is not False and dtype == torch.bfloat16 and s.scale > 0
+                and ops.latent_attention_tiled_supported(s.kv_rank, s.rot_dim))
+
+    def attend_tiled(self, qfull, out_lat, step, slot):
+        s = self.spec
+        most = step.max_kv_len if s.window is None else min(step.max_kv_len, s.window + step.max_q_len - 1)
+        ops.latent_attention_tiled(qfull, slot.kv, slot.table, step.seq_rows, step.cu_q, step.kv_len, self.sink, out_lat,
+                                   entries=step.num_seqs, max_q_len=step.max_q_len, heads=s.num_heads, rank=s.kv_rank,
+                                   rot=s.rot_dim, page_size=slot.page_size, scale=s.scale, window=s.window, max_keys=most)
 
 
 register_mixer("latent_attention", LatentAttention)

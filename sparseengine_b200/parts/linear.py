@@ -31,8 +31,9 @@ GEMV_MAX_OUT = 16384
 GEMV_MAX_ROWS = 8
 
 
-def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
-    """x [rows, in], w [out, in] → [rows, out]; CUDA tensors of one dtype only."""
+def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, activation: str | None = None) -> torch.Tensor:
+    """x [rows, in], w [out, in] → [rows, out]; CUDA tensors of one dtype only.  ``activation``: a name of
+    ``ops.ACTIVATIONS`` applied to the product (inside this library's few-row kernel, else as a kernel of its own)."""
     if not (x.is_cuda and w.is_cuda):
         raise ValueError("linear needs CUDA tensors (there is no CPU path)")
     if x.dtype != w.dtype:
@@ -43,10 +44,9 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None) ->
         # a handful of rows (decode): this library's weight-streaming kernel
         if out is None:
             out = torch.empty(x.shape[0], w.shape[0], dtype=x.dtype, device=x.device)
-        return ops.gemv(x, w, out)
-    if out is None:
-        return torch.matmul(x, w.t())
-    return torch.matmul(x, w.t(), out=out)
+        return ops.gemv(x, w, out, activation)
+    y = torch.matmul(x, w.t()) if out is None else torch.matmul(x, w.t(), out=out)
+    return y if activation is None else ops.activation_(y, activation)
 
 
 def linear32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:

@@ -1,8 +1,8 @@
 """An ungated feed-forward: ``down(act(up(x)))``.
 
-The two products are library GEMMs (or this library's few-row kernel) through
-:func:`parts.linear.linear`; the activation runs in place between them in 32-bit arithmetic
-(kernel: csrc/stream32.cu).
+The two products are library GEMMs (or this library's few-row kernel, which applies the activation
+itself) through :func:`parts.linear.linear`; after a library GEMM the activation runs in place in
+32-bit arithmetic (kernel: csrc/stream32.cu).
 """
 from __future__ import annotations
 
@@ -28,9 +28,7 @@ class PlainMLP(FeedForward):
                 "down": ParamSpec((s.hidden_size, s.intermediate_size))}
 
     def forward(self, x, step):
-        h = linear(x, self.up)
-        ops.activation_(h, self.spec.activation)
-        return linear(h, self.down)
+        return linear(linear(x, self.up, activation=self.spec.activation), self.down)
 
 
 register_feed_forward("plain_mlp", PlainMLP)

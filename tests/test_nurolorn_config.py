@@ -176,6 +176,13 @@ def test_what_a_configuration_must_have():
             load_model_spec(bad)
 
 
+def test_how_many_ctas_share_a_prompts_recurrence():
+    from sparseengine_b200.csrc import ops
+    plan = lambda *a: ops.min_gru_plan(*a, sms=148)
+    assert [plan(1, 2048, n) for n in (1, 128, 129, 512, 513, 4096)] == [1, 1, 2, 4, 8, 8]
+    assert plan(1, 4096, 2048) == 4 and plan(4, 4096, 2048) == 1 and plan(64, 64, 2048) == 4 and plan(1, 1, 10 ** 6) == 8
+
+
 def test_what_the_parts_refuse():
     from sparseengine_b200.config.specs import (AttentionSpec, LatentAttentionSpec, LayerSpec, MinGRUSpec, ModelSpec, PlainMLPSpec,
                                                 RMSNormSpec, RotarySpec, ScheduleEntry)

@@ -502,8 +502,15 @@ def test_latent_attention_with_neighbouring_pairs(rank, rot, heads, d):
         assert float((plain.double().cpu() - want).abs().max()) < bound * float(want.abs().max()), dtype
         if dtype == torch.bfloat16 and ops.latent_attention_tiled_supported(rank, rot):
             qfull = torch.empty(b.tokens, heads, D, dtype=dtype, device=dev)
-            ops.latent_q_pack(q_lat, q, inv_freq, b.positions, qfull, heads=heads, head_dim=d, rank=rank, rot=rot, rotary_dim=rot,
-                              pairing="interleaved")
+            qfull[:, :, :rank] = q_lat.transpose(0, 1)
+            # the rotated parts by the kernel of their own, and by the preparation (which writes the same page rows again)
+            ops.latent_q_rotate(q, inv_freq, b.positions, qfull, heads=heads, head_dim=d, rank=rank, rot=rot, rotary_dim=rot,
+                                pairing="interleaved")
+            again = torch.zeros_like(qfull)
+            ops.latent_prep(proj[:, cols:cols + D], None, w, inv_freq, b.positions, b.token_seq, b.seq_rows, b.table, cache, None,
+                            q_rank=0, rank=rank, rot=rot, rotary_dim=rot, eps=eps, page_size=page, pairing="interleaved",
+                            queries=(q, heads, d, again))
+            assert torch.equal(again[:, :, rank:], qfull[:, :, rank:]) and not bool(again[:, :, :rank].any())
             tiled = torch.full_like(plain, float("nan"))
             ops.latent_attention_tiled(qfull, cache, b.table, b.seq_rows, b.cu_q, b.kv_len, None, tiled, entries=b.entries,
                                        max_q_len=b.max_q_len, heads=heads, rank=rank, rot=rot, page_size=page, scale=scale)

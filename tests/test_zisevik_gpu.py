@@ -415,7 +415,8 @@ def test_tiled_latent_attention_against_the_kernel_per_token_and_head(rank, rot,
     ops.latent_attention_plain(q_lat, q, inv_freq, cache, table, seq_rows, token_seq, positions, sink, plain, heads=heads,
                                head_dim=d, rank=rank, rot=rot, rotary_dim=rot, page_size=page, scale=scale, window=window)
     qfull = torch.empty(tokens, heads, D, dtype=torch.bfloat16, device=dev)
-    ops.latent_q_pack(q_lat, q, inv_freq, positions, qfull, heads=heads, head_dim=d, rank=rank, rot=rot, rotary_dim=rot)
+    qfull[:, :, :rank] = q_lat.transpose(0, 1)
+    ops.latent_q_rotate(q, inv_freq, positions, qfull, heads=heads, head_dim=d, rank=rank, rot=rot, rotary_dim=rot)
     tiled = torch.full((tokens, heads, rank), float("nan"), dtype=torch.bfloat16, device=dev)
     ops.latent_attention_tiled(qfull, cache, table, seq_rows, cu_q, kv_len, sink, tiled, entries=entries, max_q_len=max(q_lens),
                                heads=heads, rank=rank, rot=rot, page_size=page, scale=scale, window=window)
