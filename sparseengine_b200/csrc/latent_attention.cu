@@ -39,12 +39,13 @@ __device__ __forceinline__ float rotated_element(const T* x, int i, int pos, con
 
 // The rotated parts of a token's query heads into the query rows of the tiled kernel, qfull[t, h, rank + i]; all
 // threads of the block, cos and sin of the token's angles in shared memory.
-template <typename T>
+// VEC: try 16-byte accesses (many heads); without, a thread per pair.
+template <bool VEC, typename T>
 __device__ __forceinline__ void rotate_queries(const T* q_row, int d, T* dst, int heads, int rank, int rot, int rotary_dim,
                                                int interleaved, const float* cs_t, const float* sn_t) {
     const int half = rotary_dim / 2, D = rank + rot;
     // 8 dims (neighbouring pairs) or 8 and 8 (split halves) at a time where sizes and addresses allow it
-    if (rotary_dim == rot && rot > 0 && ((interleaved ? rot : half) & 7) == 0 && (d & 7) == 0 && (rank & 7) == 0 && aligned8(q_row) &&
+    if (VEC && rotary_dim == rot && rot > 0 && ((interleaved ? rot : half) & 7) == 0 && (d & 7) == 0 && (rank & 7) == 0 && aligned8(q_row) &&
         aligned8(dst)) {
         const int items = (interleaved ? rot : half) / 8;
         for (int x = threadIdx.x; x < heads * items; x += blockDim.x) {
@@ -110,29 +111,27 @@ __global__ void latent_prep_kernel(const T* proj, int proj_stride, const T* __re
     float* sn_t = cs_sn + half;
     grid_dependency_wait();                      // the step's inputs are older, but were maybe copied just before the kernel ahead
     const int pos = positions[t];
+    const int page = write_cache ? table[(size_t)seq_rows[token_seq[t]] * table_stride + pos / page_size] : 0;
     for (int k = threadIdx.x; k < half; k += blockDim.x) sincosf((float)pos * inv_freq[k], &sn_t[k], &cs_t[k]);
     const T* row = proj + (size_t)t * proj_stride;
-    float sk = 0.f;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = to_float(row[i]); sq += v * v; }
     for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_float(row[q_rank + i]); sk += v * v; }
     const float inv_k = 1.0f / sqrtf(block_sum(sk, scratch) / (float)rank + eps);       // its barriers also publish the angles
     if (q_rank > 0) {
-        float sq = 0.f;
-        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = to_float(row[i]); sq += v * v; }
         const float inv_q = 1.0f / sqrtf(block_sum(sq, scratch) / (float)q_rank + eps);
         for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
             cq_out[(size_t)t * q_rank + i] = from_float<T>(to_float(row[i]) * inv_q * to_float(q_w[i]));
     }
     if (q != nullptr)
-        rotate_queries(q + (size_t)t * q_pitch, d, qfull + (size_t)t * heads * (rank + rot), heads, rank, rot, rotary_dim, interleaved,
+        rotate_queries<true>(q + (size_t)t * q_pitch, d, qfull + (size_t)t * heads * (rank + rot), heads, rank, rot, rotary_dim, interleaved,
                        cs_t, sn_t);
-    if (!write_cache) return;
-    const int page = table[(size_t)seq_rows[token_seq[t]] * table_stride + pos / page_size];
-    if (!page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_LATENT_PREP)) return;
+    if (!write_cache || !page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_LATENT_PREP)) return;
     const int D = rank + rot;
     T* dst = cache + ((size_t)page * page_size + pos % page_size) * D;
     for (int i = threadIdx.x; i < rank; i += blockDim.x)
         dst[i] = from_float<T>(to_float(row[q_rank + i]) * inv_k * to_float(kv_w[i]));
-    rotate_queries(row + q_rank + rank, 0, dst, 1, rank, rot, rotary_dim, interleaved, cs_t, sn_t);     // one "head"
+    rotate_queries<false>(row + q_rank + rank, 0, dst, 1, rank, rot, rotary_dim, interleaved, cs_t, sn_t);     // one "head"
 }
 
 constexpr int kLatWarps = 4;
@@ -307,7 +306,7 @@ __global__ void latent_q_rotate_kernel(const __nv_bfloat16* q, int q_pitch, int 
     for (int k = threadIdx.x; k < half; k += blockDim.x)
         sincosf((float)positions[t] * inv_freq[k], &cs_sn[half + k], &cs_sn[k]);
     __syncthreads();
-    rotate_queries(q + (size_t)t * q_pitch, d, qfull + (size_t)t * heads * (rank + rot), heads, rank, rot, rotary_dim, interleaved,
+    rotate_queries<true>(q + (size_t)t * q_pitch, d, qfull + (size_t)t * heads * (rank + rot), heads, rank, rot, rotary_dim, interleaved,
                    cs_sn, cs_sn + half);
 }
 
