@@ -94,6 +94,38 @@ __device__ __forceinline__ void rotate_queries(const T* q_row, int d, T* dst, in
 //   page row [rank, ..) = the key part, rotated by the position (rotated_element)
 // With q (rows q_pitch apart, [heads * (d + rot)]; nullptr: none) also the rotated parts of the queries into qfull
 // [tokens, heads, rank + rot].
+// The sum of squares of n elements over the block's threads (each its share), and dst = src * inv * w; 8 at a time if `vec`.
+template <typename T>
+__device__ __forceinline__ float share_of_squares(const T* src, int n, bool vec) {
+    float s = 0.f;
+    if (vec) {
+        for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+            float v[8];
+            load8(src + i, v);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) s += v[j] * v[j];
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = to_float(src[i]); s += v * v; }
+    }
+    return s;
+}
+template <typename T>
+__device__ __forceinline__ void scaled_row(const T* src, const T* __restrict__ w, float inv, T* dst, int n, bool vec) {
+    if (vec) {
+        for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+            float v[8], m[8];
+            load8(src + i, v);
+            load8(w + i, m);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = v[j] * inv * m[j];
+            store8(dst + i, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_float<T>(to_float(src[i]) * inv * to_float(w[i]));
+    }
+}
+
 template <typename T>
 __global__ void latent_prep_kernel(const T* proj, int proj_stride, const T* __restrict__ q_w, const T* __restrict__ kv_w,
                                    const float* __restrict__ inv_freq, const int* __restrict__ positions,
@@ -114,23 +146,21 @@ __global__ void latent_prep_kernel(const T* proj, int proj_stride, const T* __re
     const int page = write_cache ? table[(size_t)seq_rows[token_seq[t]] * table_stride + pos / page_size] : 0;
     for (int k = threadIdx.x; k < half; k += blockDim.x) sincosf((float)pos * inv_freq[k], &sn_t[k], &cs_t[k]);
     const T* row = proj + (size_t)t * proj_stride;
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = to_float(row[i]); sq += v * v; }
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_float(row[q_rank + i]); sk += v * v; }
+    const int D = rank + rot;
+    const bool vec = ((q_rank | rank | D) & 7) == 0 && aligned8(row) && aligned8(kv_w) && aligned8(cache) &&
+                     (q_rank == 0 || (aligned8(q_w) && aligned8(cq_out)));
+    const float sq = share_of_squares(row, q_rank, vec), sk = share_of_squares(row + q_rank, rank, vec);
     const float inv_k = 1.0f / sqrtf(block_sum(sk, scratch) / (float)rank + eps);       // its barriers also publish the angles
     if (q_rank > 0) {
         const float inv_q = 1.0f / sqrtf(block_sum(sq, scratch) / (float)q_rank + eps);
-        for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-            cq_out[(size_t)t * q_rank + i] = from_float<T>(to_float(row[i]) * inv_q * to_float(q_w[i]));
+        scaled_row(row, q_w, inv_q, cq_out + (size_t)t * q_rank, q_rank, vec);
     }
     if (q != nullptr)
         rotate_queries<true>(q + (size_t)t * q_pitch, d, qfull + (size_t)t * heads * (rank + rot), heads, rank, rot, rotary_dim, interleaved,
                        cs_t, sn_t);
     if (!write_cache || !page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_LATENT_PREP)) return;
-    const int D = rank + rot;
     T* dst = cache + ((size_t)page * page_size + pos % page_size) * D;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x)
-        dst[i] = from_float<T>(to_float(row[q_rank + i]) * inv_k * to_float(kv_w[i]));
+    scaled_row(row + q_rank, kv_w, inv_k, dst, rank, vec);
     rotate_queries<false>(row + q_rank + rank, 0, dst, 1, rank, rot, rotary_dim, interleaved, cs_t, sn_t);     // one "head"
 }
 
