@@ -9,7 +9,7 @@ pages per kind of layer, and fixed-size per-request state slots.
   ``i*page_size .. (i+1)*page_size-1`` in every cache layer of the group.
 * A request is **admitted** (gets a row and zeroed state slots), **reserves** pages for
   its next tokens before a step (all groups or none), **commits** them after the step
-  (a windowed group then gives back the pages no later query can see; pages that hold the first
+  (a group with a window or a chunk then gives back the pages no later query can see; pages that hold the first
   ``keep_first`` positions of a group that keeps them are never given back early) and is
   **released** when it ends (everything returns to the pools).
 * **State slots**: ``state[i][row]`` is a tensor of fixed shape per request for schedule
@@ -194,17 +194,17 @@ class CacheManager:
         r.reserved += n_tokens
 
     def commit(self, seq_id, n_tokens: int) -> None:
-        """The step wrote ``n_tokens`` of the reserved tokens.  A windowed group gives
-        back every page whose positions no later query can see."""
+        """The step wrote ``n_tokens`` of the reserved tokens.  A group with a window
+        or a chunk gives back every page whose positions no later query can see."""
         r = self._requests[seq_id]
         if n_tokens > r.reserved:
             raise ValueError("commit of more tokens than were reserved")
         r.reserved -= n_tokens
         r.length += n_tokens
         for gi, g in enumerate(self.groups):
-            if g.window is None:
+            if not g.request.bounded:
                 continue
-            first_needed = max(0, r.length - g.window + 1)     # the next query's oldest key
+            first_needed = g.request.first_visible(r.length)   # the next query's oldest key
             keep = getattr(g.request, "keep_first", 0)         # positions below it stay visible to every later query
             dead = [idx for idx in r.pages[gi] if (idx + 1) * self.page_size <= first_needed
                     and idx * self.page_size >= keep]

@@ -91,10 +91,12 @@ class AttentionSpec:
     scale: float = 1.0
     # None | "whole_projection" (one root mean square over all heads, a weight per column) | "per_head" (one per
     # head, a weight of head_dim elements shared by the heads; needs prep="general") | "per_head_unit" (one per
-    # head, no weight; needs prep="general")
+    # head, no weight, of the rotated head; needs prep="general")
     qk_norm: Optional[str] = None
     qk_norm_eps: float = 1e-6
     window: Optional[int] = None      # keys p-window+1..p; None = all keys
+    # instead of a window: keys of the query's own chunk, floor(j / chunk) = floor(p / chunk), counted from position 0
+    chunk: Optional[int] = None
     position: Optional[Any] = None    # a position-encoding spec (e.g. RotarySpec)
     # "rotary": the fused norm + rotation kernel (values as wide as keys).  "general": no rotation;
     # the fields below apply, and norms and temperature are computed in 32-bit and rounded once.
@@ -103,7 +105,7 @@ class AttentionSpec:
     # (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)
     q_temperature: Optional[tuple] = None
     own_kv: bool = True               # False: no key/value projections; the layer attends over another's cache
-    # The fields below need prep="general", which then also rotates (``position``: split halves, no factor).
+    # The fields below need prep="general", which then also rotates (``position``: split halves or neighbours).
     score_softcap: Optional[float] = None   # c: the scaled score becomes c * tanh(score / c)
     # "zero": a key of score 0 that has no value joins the softmax: p_j = exp(s_j) / (1 + sum exp(s_j)).
     # "learned": the same with a learned logit per head (parameter ``sink``) in place of 0, unscaled.
@@ -114,12 +116,13 @@ class AttentionSpec:
     # a distance bias: one slope per query head; the scaled score of query position i and key position j loses
     # slope * (i - j)
     distance_slopes: Optional[tuple] = None
-    # biases on the q, k, v rows of the packed projection (parameter ``qkv_bias``) and on the output projection
-    # (``o_bias``); needs prep="general"
+    # biases on the q, k, v rows of the packed projection (parameter ``qkv_bias``) and, unless ``output_bias`` says
+    # otherwise, on the output projection (``o_bias``); needs prep="general"
     bias: bool = False
-    # the concatenated heads are multiplied by sigmoid(W_g x) before the output projection; W_g's
-    # rows follow the values' in the packed projection
-    output_gate: bool = False
+    output_bias: Optional[bool] = None      # None: as ``bias``
+    # the concatenated heads are multiplied by sigmoid(W_g x) before the output projection; W_g's rows follow the
+    # values' in the packed projection.  True (or "element"): one number per output element; "head": one per head
+    output_gate: Any = False
     # "first": this layer's values (of this step's tokens) are kept for the layers after it.
     # "blend": the values become (1 - m) v + m v_first with a learned number m, before they are cached.
     # Both kinds own the parameter ``v_mix`` (a "first" layer does not use it).
@@ -189,13 +192,16 @@ class MatrixMemorySpec:
 
 @dataclass(frozen=True)
 class ParallelMixerSpec:
-    """Mixers side by side on the same input: the result is ``sum_i scales[i] * branch_i(x)``.  At most one
-    branch may ask for pages and at most one for a state slot."""
+    """Mixers side by side on the same input: the result is ``sum_i scales[i] * branch_i(x)``, or with
+    ``output_norms`` ``sum_i scales[i] * rms(branch_i(x)) * w_i`` (each branch's result over its root mean square, times
+    a weight, before the sum).  At most one branch may ask for pages and at most one for a state slot."""
     kind: str = "parallel"
     hidden_size: int = 0
     branches: tuple = ()              # mixer specs
     scales: tuple = ()                # one factor per branch
     names: tuple = ()                 # a name per branch: its parameters are "<name>_<parameter>"
+    output_norms: bool = False        # parameters "<name>_out_norm"
+    norm_eps: float = 1e-6
 
 
 @dataclass(frozen=True)
@@ -242,9 +248,11 @@ class LatentAttentionSpec:
 @dataclass(frozen=True)
 class RetentionSpec:
     """Linear attention with one fixed decay per head: ``S <- decay S + k v^T``, ``o = S^T q``, no
-    softmax or denominator.  q and k are rotated (``position``), k is scaled by ``head_dim ** -0.5``
+    softmax or denominator.  q and k are rotated (``position``), k is scaled by ``k_scale`` (default ``head_dim ** -0.5``)
     after the rotation; each head's ``o`` is divided by its root mean square (no weight), multiplied
-    by ``silu(gate)`` and projected."""
+    by ``silu(gate)`` and projected.  ``activation="silu"``: q, k and v are silu of their projections (lightning
+    attention).  ``output_norm="joint"``: the concatenated heads are divided by one root mean square, multiplied by a
+    weight per column (parameter ``norm_w``) and by ``sigmoid(gate)``."""
     kind: str = "retention"
     hidden_size: int = 0
     num_heads: int = 0
@@ -253,6 +261,9 @@ class RetentionSpec:
     decays: tuple = ()                # one per head
     position: Optional[Any] = None    # RotarySpec, split-half pairing
     norm_eps: float = 1e-6
+    activation: Optional[str] = None  # None | "silu"
+    k_scale: Optional[float] = None   # None: head_dim ** -0.5
+    output_norm: str = "per_head"     # "per_head" (no weight, silu gate) | "joint" (weight, sigmoid gate)
 
 
 @dataclass(frozen=True)
@@ -280,7 +291,8 @@ class MoESpec:
     renormalize: bool = True
     routed_scale: float = 1.0
     # "silu": silu(gate) * up.  "clamped_swiglu": g * sigmoid(activation_alpha * g) * (u + 1) with
-    # g = min(gate, activation_limit) and u = clamp(up, -activation_limit, activation_limit).
+    # g = min(gate, activation_limit) and u = clamp(up, -activation_limit, activation_limit).  "gelu_tanh": gelu(gate) *
+    # up with gelu in its tanh form.
     activation: str = "silu"
     activation_limit: float = 0.0
     activation_alpha: float = 1.702
@@ -338,6 +350,9 @@ class LayerSpec:
     # "sublayer_norm": x <- x + norm(mixer(x)), x <- x + norm(ff(x)) over a 32-bit stream: the norms
     # sit on the sublayers' outputs and the sublayers read x itself; the feed-forward (with its
     # norm) may be None
+    # "sandwich_norm": x <- x + norm_b(mixer(norm_a(x))), x <- x + norm_b(ff(norm_a(x))) over a 32-bit stream: RMS norms
+    # before and after each sublayer; extra["mixer_post_norm"] and extra["feed_forward_post_norm"] are the latter's specs;
+    # the feed-forward (with its norms) may be None
     residual_scale: float = 1.0
     extra: dict = field(default_factory=dict)       # part name -> spec, for arrangements with more parts
     # part-local parameter name -> tuple[Source, ...]; keys are "<part>.<param>" with

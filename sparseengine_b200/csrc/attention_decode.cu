@@ -11,8 +11,10 @@
 // src/sparseengine/kernels/triton/flash_decoding_stage2.py:27-45): scores and softmax in
 // 32-bit, probabilities rounded to bfloat16 before they multiply V, the output rounded once.
 //
-// Any page size; query/key head sizes 64 and 128, value head sizes 32, 64 and 128 (others use the
-// plain kernel); a window is honoured, with or without first keys that stay visible.  A page holds the keys [kv head][slot][D] and then the values
+// Any page size; query/key and value head sizes that are multiples of 8 up to 128 (others use the plain
+// kernel): tiles have 64 or 128 query/key columns and 32, 64 or 128 value columns, and a head size between
+// them lies in the next wider tile, the columns beyond it zero.  A window (with or without first keys that
+// stay visible) or a chunk (first_visible) is honoured.  A page holds the keys [kv head][slot][D] and then the values
 // [kv head][slot][DV].  The softmax's options (a cap on the scores, a sink, an output gate, a distance bias)
 // are those of mma_util.cuh's SoftmaxOptions; the sink joins once, where the last sum is taken (here
 // for one split, in the second kernel for several), and the gate where the output is rounded.
@@ -32,14 +34,16 @@ constexpr int kThreads = 32 * kWarps;
 
 using namespace se::mma;
 
-template <int D, int DV>
+template <int D, int DV, bool PAD>
 __global__ void __launch_bounds__(kThreads)
 attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // written by the kernel before this one: no __restrict__ (see the wait below)
                    const int* __restrict__ table, int table_stride, const int* __restrict__ seq_rows,
                    const int* __restrict__ token_seq, const int* __restrict__ positions,
                    __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int hq,
                    int hkv, int page_size, float scale_log2, int window, int splits, int keys_per_split,
-                   int num_pages, int* __restrict__ error, const SoftmaxOptions opt) {
+                   int num_pages, int* __restrict__ error, const SoftmaxOptions opt, int d_run, int dv_run) {
+    // the head sizes in memory; D and DV are those of the tiles, whose columns beyond them stay zero
+    const int d_real = PAD ? d_run : D, dv_real = PAD ? dv_run : DV;
     constexpr int kTileBytes = kTileKeys * D * 2;    // one K tile
     constexpr int kStageBytes = kTileKeys * (D + DV) * 2;    // a K tile and a V tile
     extern __shared__ __align__(128) uint8_t smem[];
@@ -57,15 +61,15 @@ attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // w
     const int pos = positions[t];
     // The keys a token sees, in the order they are visited: the kept first ones that lie before the window,
     // then the window's.  ks, ke and the tiles count in that order; key_of gives a place's position.
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_visible(pos, window);
     const int kept = min(opt.keep_first, lo);
     const int ks = split * keys_per_split;
     const int ke = min(kept + pos + 1 - lo, ks + keys_per_split);
     auto key_of = [&](int n) { return n < kept ? n : lo + n - kept; };
     const int* row_table = table + (size_t)seq_rows[token_seq[t]] * table_stride;
-    const size_t page_elems = (size_t)hkv * page_size * (D + DV);
-    const size_t head_off = (size_t)kvh * page_size * D;
-    const size_t v_off = (size_t)hkv * page_size * D + (size_t)kvh * page_size * DV;
+    const size_t page_elems = (size_t)hkv * page_size * (d_real + dv_real);
+    const size_t head_off = (size_t)kvh * page_size * d_real;
+    const size_t v_off = (size_t)hkv * page_size * d_real + (size_t)kvh * page_size * dv_real;
 
     float o[DV / 8][4];
 #pragma unroll
@@ -76,13 +80,15 @@ attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // w
 
     // Rows [64][DIM] of a tile: a thread copies chunk (tid % chunks) of rows tid / chunks + k * (kThreads / chunks).
     // The rows' addresses are looked up first (independent loads), so that no table load sits
-    // between the asynchronous copies.  `off`: where the head's rows start in a page; DIM elements a row.
-    auto load_rows = [&](auto dim_tag, uint8_t* dst, int base, size_t off) {
+    // between the asynchronous copies.  `off`: where the head's rows start in a page; `dim` elements a
+    // row in memory, DIM in the tile.
+    auto load_rows = [&](auto dim_tag, int dim, uint8_t* dst, int base, size_t off) {
         constexpr int DIM = decltype(dim_tag)::value;
         constexpr int kChunks = DIM / 8;                 // 16-byte chunks per row
         constexpr int kRowStep = kThreads / kChunks, kIters = kTileKeys / kRowStep;
         static_assert(kThreads % kChunks == 0 && kTileKeys % kRowStep == 0, "tile copy mapping");
         const int c = threadIdx.x % kChunks, r0t = threadIdx.x / kChunks;
+        const bool col_ok = !PAD || c * 8 < dim;
         const __nv_bfloat16* srcs[kIters];
         bool page_ok[kIters];
 #pragma unroll
@@ -92,19 +98,19 @@ attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // w
             const int page = row_table[jj / page_size];
             // an entry that names no page of the pool is not followed: its rows are zero-filled
             page_ok[k] = page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_ATTN_DECODE);
-            srcs[k] = cache + (size_t)(page_ok[k] ? page : 0) * page_elems + off + (size_t)(jj % page_size) * DIM + c * 8;
+            srcs[k] = cache + (size_t)(page_ok[k] ? page : 0) * page_elems + off + (size_t)(jj % page_size) * dim + (col_ok ? c * 8 : 0);
         }
 #pragma unroll
         for (int k = 0; k < kIters; ++k) {
             const int r = r0t + k * kRowStep;
-            cp_async16(smem_u32(dst) + tile_off<DIM>(r, c), srcs[k], base + r < ke && page_ok[k]);
+            cp_async16(smem_u32(dst) + tile_off<DIM>(r, c), srcs[k], base + r < ke && page_ok[k] && col_ok);
         }
     };
     auto load_tile = [&](int tile, int stage) {
         uint8_t* kbase = smem + (size_t)stage * kStageBytes;
         const int base = ks + tile * kTileKeys;
-        load_rows(std::integral_constant<int, D>{}, kbase, base, head_off);
-        load_rows(std::integral_constant<int, DV>{}, kbase + kTileBytes, base, v_off);
+        load_rows(std::integral_constant<int, D>{}, d_real, kbase, base, head_off);
+        load_rows(std::integral_constant<int, DV>{}, dv_real, kbase + kTileBytes, base, v_off);
     };
 
     // Where the step's inputs are older than the kernel before this one (the one that writes the
@@ -116,16 +122,17 @@ attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // w
     // Q fragments (A operand, 16 rows x D): rows g and g+8 of this lane
     uint32_t qa[D / 16][4];
     {
-        const __nv_bfloat16* q0 = q + ((size_t)t * hq + head0 + g) * D;
-        const __nv_bfloat16* q1 = q + ((size_t)t * hq + head0 + g + 8) * D;
+        const __nv_bfloat16* q0 = q + ((size_t)t * hq + head0 + g) * d_real;
+        const __nv_bfloat16* q1 = q + ((size_t)t * hq + head0 + g + 8) * d_real;
         const bool v0 = g < rows_valid, v1 = g + 8 < rows_valid;
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
             const int c = kk * 16 + 2 * t4;
-            qa[kk][0] = v0 ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
-            qa[kk][1] = v1 ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
-            qa[kk][2] = v0 ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
-            qa[kk][3] = v1 ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
+            const bool lo_ok = !PAD || kk * 16 < d_real, hi_ok = !PAD || kk * 16 + 8 < d_real;      // head sizes are multiples of 8
+            qa[kk][0] = v0 && lo_ok ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
+            qa[kk][1] = v1 && lo_ok ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
+            qa[kk][2] = v0 && hi_ok ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
+            qa[kk][3] = v1 && hi_ok ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
         }
     }
 
@@ -242,8 +249,8 @@ attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // w
         r_hi[0] = o[i][2]; r_hi[1] = o[i][3];
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < rows_valid * DV; i += kThreads) {
-        const int r = i / DV, d = i % DV;
+    for (int i = threadIdx.x; i < rows_valid * dv_real; i += kThreads) {
+        const int r = i / dv_real, d = i % dv_real;
         float mt = -INFINITY;
 #pragma unroll
         for (int w = 0; w < kWarps; ++w) mt = fmaxf(mt, sm_m[w * 16 + r]);
@@ -260,11 +267,11 @@ attn_decode_kernel(const __nv_bfloat16* q, const __nv_bfloat16* cache,      // w
             // the sink's term 2^(0 - mt): it grows beyond the type only where the keys hold nothing (the output is 0 then)
             if (opt.sink) lt += exp2f(sink_log2(opt, head) - mt * scale_log2);
             float v = acc / lt;
-            if (opt.gate != nullptr) v = gated(v, opt.gate + (size_t)t * opt.gate_pitch + (size_t)head * DV + d);
-            out[((size_t)t * hq + head) * DV + d] = __float2bfloat16_rn(v);
+            if (opt.gate != nullptr) v = gated(v, gate_of(opt, t, head, dv_real) + (opt.gate_per_head ? 0 : d));
+            out[((size_t)t * hq + head) * dv_real + d] = __float2bfloat16_rn(v);
         } else {
             const size_t pidx = ((size_t)t * hq + head) * splits + split;
-            part_o[pidx * DV + d] = acc;
+            part_o[pidx * dv_real + d] = acc;
             if (d == 0) {
                 part_ml[pidx * 2] = mt == -INFINITY ? -INFINITY : mt * scale_log2;
                 part_ml[pidx * 2 + 1] = lt;
@@ -291,16 +298,16 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
         }
         if (opt.sink) lt += exp2f(sink_log2(opt, (int)(th % hq)) - mt);
         float v = acc / lt;
-        if (opt.gate != nullptr) v = gated(v, opt.gate + (th / hq) * opt.gate_pitch + (th % hq) * d + i);
+        if (opt.gate != nullptr) v = gated(v, gate_of(opt, th / hq, th % hq, d) + (opt.gate_per_head ? 0 : i));
         out[th * d + i] = __float2bfloat16_rn(v);
     }
 }
 
-template <int D, int DV>
+template <int D, int DV, bool PAD>
 static int launch(const void* q, const void* cache, const int* table, int table_stride, const int* seq_rows,
                   const int* token_seq, const int* positions, void* out, float* part_o, float* part_ml, int tokens,
                   int hq, int hkv, int page_size, float scale, int window, int splits, int keys_per_split,
-                  int num_pages, int* error, int settled, const SoftmaxOptions& opt, cudaStream_t stream) {
+                  int num_pages, int* error, int settled, const SoftmaxOptions& opt, int d, int dv, cudaStream_t stream) {
     const int group = hq / hkv;
     const int gtiles = (group + 15) / 16;
     const size_t stage_smem = (size_t)kStages * kTileKeys * (D + DV) * 2;
@@ -308,19 +315,19 @@ static int launch(const void* q, const void* cache, const int* table, int table_
     const size_t smem = stage_smem > merge_smem ? stage_smem : merge_smem;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<D, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<D, DV, PAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(tokens, hkv * gtiles, splits);
     cudaError_t e = SE_LAUNCH_DEPENDENT_IF(
-        settled != 0, "attn", attn_decode_kernel<D, DV>, grid, dim3(kThreads), smem, stream, (const __nv_bfloat16*)q,
+        settled != 0, "attn", attn_decode_kernel<D, DV, PAD>, grid, dim3(kThreads), smem, stream, (const __nv_bfloat16*)q,
         (const __nv_bfloat16*)cache, table, table_stride, seq_rows, token_seq, positions, (__nv_bfloat16*)out, part_o,
-        part_ml, hq, hkv, page_size, scale * 1.4426950408889634f, window, splits, keys_per_split, num_pages, error, opt);
+        part_ml, hq, hkv, page_size, scale * 1.4426950408889634f, window, splits, keys_per_split, num_pages, error, opt, d, dv);
     if (e == cudaSuccess) e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
     if (splits > 1) {
-        attn_combine_kernel<<<tokens * hq, 128, 0, stream>>>(part_o, part_ml, (__nv_bfloat16*)out, DV, splits, hq, opt);
+        attn_combine_kernel<<<tokens * hq, 128, 0, stream>>>(part_o, part_ml, (__nv_bfloat16*)out, dv, splits, hq, opt);
         e = cudaGetLastError();
     }
     return (int)e;
@@ -330,11 +337,11 @@ static int launch(const void* q, const void* cache, const int* table, int table_
 }  // namespace se
 
 extern "C" int se_attn_decode_supported(int head_dim, int hq, int hkv) {
-    return ((head_dim == 64 || head_dim == 128) && hkv > 0 && hq % hkv == 0) ? 1 : 0;
+    return (head_dim > 0 && head_dim <= 128 && head_dim % 8 == 0 && hkv > 0 && hq % hkv == 0) ? 1 : 0;
 }
 // the value head sizes the kernel takes beside a query/key head size it takes
 extern "C" int se_attn_decode_value_dim_supported(int v_head_dim) {
-    return (v_head_dim == 32 || v_head_dim == 64 || v_head_dim == 128) ? 1 : 0;
+    return (v_head_dim > 0 && v_head_dim <= 128 && v_head_dim % 8 == 0) ? 1 : 0;
 }
 
 // part_o: float [tokens, hq, splits, v_head_dim]; part_ml: float [tokens, hq, splits, 2] (unused when splits == 1).
@@ -349,24 +356,33 @@ extern "C" int se_attn_decode(const void* q, const void* cache, const int* table
                               float* part_o, float* part_ml, int tokens, int hq, int hkv, int head_dim, int v_head_dim,
                               int page_size, float scale, int window, int splits, int keys_per_split, int num_pages,
                               int* error, int settled, float softcap, int sink, const void* gate, int gate_pitch,
-                              const float* sink_logits, int keep_first, const float* slopes, cudaStream_t stream) {
+                              const float* sink_logits, int keep_first, const float* slopes, int gate_per_head,
+                              cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (!se_attn_decode_supported(head_dim, hq, hkv) || !se_attn_decode_value_dim_supported(v_head_dim) || splits < 1 ||
         keys_per_split <= 0 || keys_per_split % 64)
         return SE_ERR_UNSUPPORTED;
     if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) return SE_ERR_ARGUMENT;
-    if (softcap < 0.f || !(scale > 0.f) || (gate != nullptr && gate_pitch < hq * v_head_dim) || keep_first < 0)
+    if (softcap < 0.f || !(scale > 0.f) || (gate != nullptr && gate_pitch < (gate_per_head ? hq : hq * v_head_dim)) || keep_first < 0)
         return SE_ERR_ARGUMENT;
     const se::mma::SoftmaxOptions opt{softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f,
                                       sink || sink_logits != nullptr, (const __nv_bfloat16*)gate, gate_pitch, sink_logits,
-                                      window > 0 ? keep_first : 0, slopes, 1.f / scale};
+                                      window > 0 ? keep_first : 0, slopes, 1.f / scale, gate_per_head};
+    // tiles of 64 or 128 query/key columns and 32, 64 or 128 value columns; head sizes between them in the next wider tile
+    const int dt = head_dim <= 64 ? 64 : 128, dvt = v_head_dim <= 32 ? 32 : v_head_dim <= 64 ? 64 : 128;
+    const bool pad = dt != head_dim || dvt != v_head_dim;
+#define SE_DECODE_LAUNCH(DQ, DVAL, PAD)                                                                                 \
+    return se::dec::launch<DQ, DVAL, PAD>(q, cache, table, table_stride, seq_rows, token_seq, positions, out, part_o,   \
+                                          part_ml, tokens, hq, hkv, page_size, scale, window, splits, keys_per_split,   \
+                                          num_pages, error, settled, opt, head_dim, v_head_dim, stream)
 #define SE_DECODE_CASE(DQ, DVAL)                                                                                        \
-    if (head_dim == DQ && v_head_dim == DVAL)                                                                           \
-        return se::dec::launch<DQ, DVAL>(q, cache, table, table_stride, seq_rows, token_seq, positions, out, part_o,   \
-                                         part_ml, tokens, hq, hkv, page_size, scale, window, splits, keys_per_split,    \
-                                         num_pages, error, settled, opt, stream);
+    if (dt == DQ && dvt == DVAL) {                                                                                      \
+        if (pad) SE_DECODE_LAUNCH(DQ, DVAL, true);                                                                      \
+        SE_DECODE_LAUNCH(DQ, DVAL, false);                                                                              \
+    }
     SE_DECODE_CASE(64, 64) SE_DECODE_CASE(128, 128) SE_DECODE_CASE(64, 32) SE_DECODE_CASE(64, 128)
     SE_DECODE_CASE(128, 64) SE_DECODE_CASE(128, 32)
+#undef SE_DECODE_LAUNCH
 #undef SE_DECODE_CASE
     return SE_ERR_UNSUPPORTED;
 }

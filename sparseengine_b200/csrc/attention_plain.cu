@@ -3,13 +3,14 @@
 // sizes the tensor-core kernels refuse.
 //
 // score = q·k * scale; query at position p sees keys max(0, p-window+1)..p of its own
-// request (window 0 = all keys); softmax state and accumulators in 32-bit; the
+// request (window 0 = all keys, window -n = the keys of p's own chunk of n positions); softmax state and accumulators in 32-bit; the
 // probability is rounded to the activation type before it multiplies V; the output is
 // rounded once.  The value head size `dv` may differ from the query/key size `d`: a page holds
 // the keys [kv head][slot][d] and then the values [kv head][slot][dv].
 // Options: `softcap` c > 0 caps the scaled score, s <- c tanh(s / c); `sink` adds a key of score 0
 // that has no value (one more term, exp(0), in the softmax's denominator); `gate` (with its row
-// pitch) multiplies the output element by element with sigmoid(gate[t][h * dv + i]); `sink_logits`
+// pitch) multiplies the output element by element with sigmoid(gate[t][h * dv + i]), or with `gate_per_head` a
+// whole head with sigmoid(gate[t][h]); `sink_logits`
 // (one per query head) puts a learned logit in the place of the sink's 0, unscaled; `keep_first` n > 0
 // (with a window) keeps keys 0..n-1 visible beside the window's; `slopes` (one per query head) takes
 // slope * (i - j) off the score of query position i and key position j.  Reference: src/sparseengine/kernels/triton/context_flashattention_nopad.py:92-127,
@@ -34,13 +35,13 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
                                              int* __restrict__ error, float softcap, int sink,
                                              const T* __restrict__ gate, int gate_pitch,
                                              const float* __restrict__ sink_logits, int keep_first,
-                                             const float* __restrict__ slopes) {
+                                             const float* __restrict__ slopes, int gate_per_head) {
     const int t = blockIdx.x, h = blockIdx.y;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int kvh = h / (hq / hkv);
     const int pos = positions[t];
     const int* row_table = table + (size_t)seq_rows[token_seq[t]] * table_stride;
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_visible(pos, window);
     const size_t page_elems = (size_t)hkv * page_size * (d + dv);
     const size_t v_off = (size_t)hkv * page_size * d + (size_t)kvh * page_size * dv;
     const size_t head_off = (size_t)kvh * page_size * d;
@@ -105,7 +106,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, const T* _
 #pragma unroll
         for (int w = 0; w < kAttnWarps; ++w) o += sm[w] == -INFINITY ? 0.f : sacc[w][dim] * expf(sm[w] - mt);
         o /= lt;
-        if (gate != nullptr) o /= 1.f + expf(-to_float(gate[(size_t)t * gate_pitch + (size_t)h * dv + dim]));
+        if (gate != nullptr) o /= 1.f + expf(-to_float(gate[(size_t)t * gate_pitch + (gate_per_head ? (size_t)h : (size_t)h * dv + dim)]));
         op[dim] = from_float<T>(o);
     }
 }
@@ -116,10 +117,12 @@ extern "C" int se_paged_attention_plain(const void* q, const void* cache, const 
                                         const int* seq_rows, const int* token_seq, const int* positions, void* out,
                                         int tokens, int hq, int hkv, int d, int dv, int page_size, float scale, int window,
                                         int num_pages, int* error, float softcap, int sink, const void* gate, int gate_pitch,
-                                        const float* sink_logits, int keep_first, const float* slopes, int dtype, cudaStream_t stream) {
+                                        const float* sink_logits, int keep_first, const float* slopes, int gate_per_head, int dtype,
+                                        cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (softcap < 0.f || (gate != nullptr && gate_pitch < hq * dv) || keep_first < 0) return SE_ERR_ARGUMENT;
+    if (softcap < 0.f || (gate != nullptr && gate_pitch < (gate_per_head ? hq : hq * dv)) || keep_first < 0) return SE_ERR_ARGUMENT;
     if (sink_logits != nullptr) sink = 1;
+    if (window <= 0) keep_first = 0;
     if (d > 32 * se::kMaxDimPerLane || d <= 0 || dv > 32 * se::kMaxDimPerLane || dv <= 0 || hkv <= 0 || hq % hkv)
         return SE_ERR_UNSUPPORTED;
     dim3 grid(tokens, hq);
@@ -127,6 +130,6 @@ extern "C" int se_paged_attention_plain(const void* q, const void* cache, const 
         se::paged_attention_plain_kernel<T><<<grid, 32 * se::kAttnWarps, 0, stream>>>(
             (const T*)q, (const T*)cache, table, table_stride, seq_rows, token_seq, positions, (T*)out, hq, hkv, d, dv,
             page_size, scale, window, num_pages, error, softcap, sink, (const T*)gate, gate_pitch,
-            sink_logits, keep_first, slopes));
+            sink_logits, keep_first, slopes, gate_per_head));
     SE_LAUNCH_CHECK();
 }

@@ -11,8 +11,10 @@
 // cache before this kernel runs.  Reference arithmetic:
 // src/sparseengine/kernels/triton/context_flashattention_nopad.py:92-127.
 //
-// Any page size; query/key head sizes 64 and 128, value head sizes 32, 64 and 128 (others use the
-// plain kernel): a page holds the keys [kv head][slot][D] and then the values [kv head][slot][DV].
+// Any page size; query/key and value head sizes that are multiples of 8 up to 128 (others use the plain
+// kernel): tiles have 64 or 128 query/key columns and 32, 64 or 128 value columns, and a head size between
+// them lies in the next wider tile, the columns beyond it zero.  Instead of a window, a chunk may bound
+// the keys (first_visible).  A page holds the keys [kv head][slot][D] and then the values [kv head][slot][DV].
 // The softmax's options (a cap on the scores, a sink, an output gate, a distance bias) are those of
 // mma_util.cuh's SoftmaxOptions.  A block-table entry outside [0, num_pages) is not followed: its
 // rows are zero-filled and a code goes to the error word.
@@ -31,13 +33,15 @@ constexpr int kThreads = 32 * kWarps;
 
 using namespace se::mma;
 
-template <int D, int DV>
+template <int D, int DV, bool PAD>
 __global__ void __launch_bounds__(kThreads)
 attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache,
                     const int* __restrict__ table, int table_stride, const int* __restrict__ seq_rows,
                     const int* __restrict__ cu_q, const int* __restrict__ kv_len, __nv_bfloat16* __restrict__ out,
                     int hq, int hkv, int page_size, float scale_log2, int window, int num_pages,
-                    int* __restrict__ error, const SoftmaxOptions opt) {
+                    int* __restrict__ error, const SoftmaxOptions opt, int d_run, int dv_run) {
+    // the head sizes in memory; D and DV are those of the tiles, whose columns beyond them stay zero
+    const int d_real = PAD ? d_run : D, dv_real = PAD ? dv_run : DV;
     constexpr int kTileBytes = kTileKeys * D * 2;             // one K tile
     constexpr int kStageBytes = kTileKeys * (D + DV) * 2;     // a K tile and a V tile
     extern __shared__ __align__(128) uint8_t smem[];
@@ -73,7 +77,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     const int last_row = min(row_base + kTileRows, total_rows) - 1;
     const int max_pos = q_start + last_row / group;
     const int first_pos = q_start + row_base / group;
-    const int k_lo = window > 0 ? max(0, first_pos - window + 1) : 0;
+    const int k_lo = first_visible(first_pos, window);
     const int k_begin = (k_lo / kTileKeys) * kTileKeys;
     const int k_end = max_pos + 1;
     // first keys that stay visible: those before the CTA's window come as tiles of their own, ahead of the window's
@@ -83,21 +87,22 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     const int num_tiles = kept_tiles + (k_end - k_begin + kTileKeys - 1) / kTileKeys;
 
     const int* row_table = table + (size_t)seq_rows[entry] * table_stride;
-    const size_t page_elems = (size_t)hkv * page_size * (D + DV);
-    const size_t head_off = (size_t)kvh * page_size * D;
-    const size_t v_off = (size_t)hkv * page_size * D + (size_t)kvh * page_size * DV;
+    const size_t page_elems = (size_t)hkv * page_size * (d_real + dv_real);
+    const size_t head_off = (size_t)kvh * page_size * d_real;
+    const size_t v_off = (size_t)hkv * page_size * d_real + (size_t)kvh * page_size * dv_real;
 
     uint32_t qa[D / 16][4];
     {
-        const __nv_bfloat16* q0 = q + ((size_t)tok[0] * hq + head[0]) * D;
-        const __nv_bfloat16* q1 = q + ((size_t)tok[1] * hq + head[1]) * D;
+        const __nv_bfloat16* q0 = q + ((size_t)tok[0] * hq + head[0]) * d_real;
+        const __nv_bfloat16* q1 = q + ((size_t)tok[1] * hq + head[1]) * d_real;
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
             const int c = kk * 16 + 2 * t4;
-            qa[kk][0] = valid[0] ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
-            qa[kk][1] = valid[1] ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
-            qa[kk][2] = valid[0] ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
-            qa[kk][3] = valid[1] ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
+            const bool lo_ok = !PAD || kk * 16 < d_real, hi_ok = !PAD || kk * 16 + 8 < d_real;      // head sizes are multiples of 8
+            qa[kk][0] = valid[0] && lo_ok ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
+            qa[kk][1] = valid[1] && lo_ok ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
+            qa[kk][2] = valid[0] && hi_ok ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
+            qa[kk][3] = valid[1] && hi_ok ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
         }
     }
     float o[DV / 8][4];
@@ -108,19 +113,21 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     float slope[2];                   // the distance bias of the row's head per token, in raw score units
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-        lo[h] = window > 0 ? max(0, pos[h] - window + 1) : 0;
+        lo[h] = first_visible(pos[h], window);
         slope[h] = raw_slope(opt, head[h]);
     }
 
     // Rows [64][DIM] of a tile: a thread copies chunk (tid % chunks) of rows tid / chunks + k * (kThreads / chunks).
     // The rows' addresses are looked up first (independent loads), so that no table load sits
-    // between the asynchronous copies.  `off`: where the head's rows start in a page; DIM elements a row.
-    auto load_rows = [&](auto dim_tag, uint8_t* dst, int base, size_t off, int k_lo, int k_end) {
+    // between the asynchronous copies.  `off`: where the head's rows start in a page; `dim` elements a
+    // row in memory, DIM in the tile.
+    auto load_rows = [&](auto dim_tag, int dim, uint8_t* dst, int base, size_t off, int k_lo, int k_end) {
         constexpr int DIM = decltype(dim_tag)::value;
         constexpr int kChunks = DIM / 8;
         constexpr int kRowStep = kThreads / kChunks, kIters = kTileKeys / kRowStep;
         static_assert(kThreads % kChunks == 0 && kTileKeys % kRowStep == 0, "tile copy mapping");
         const int c = threadIdx.x % kChunks, r0t = threadIdx.x / kChunks;
+        const bool col_ok = !PAD || c * 8 < dim;
         const __nv_bfloat16* srcs[kIters];
         bool page_ok[kIters];
 #pragma unroll
@@ -132,12 +139,12 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
             const int jj = min(max(j, k_lo), k_end - 1);
             const int page = row_table[jj / page_size];
             page_ok[k] = page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_ATTN_PREFILL);
-            srcs[k] = cache + (size_t)(page_ok[k] ? page : 0) * page_elems + off + (size_t)(jj % page_size) * DIM + c * 8;
+            srcs[k] = cache + (size_t)(page_ok[k] ? page : 0) * page_elems + off + (size_t)(jj % page_size) * dim + (col_ok ? c * 8 : 0);
         }
 #pragma unroll
         for (int k = 0; k < kIters; ++k) {
             const int r = r0t + k * kRowStep;
-            const bool ok = base + r < k_end && base + r >= k_lo && page_ok[k];
+            const bool ok = base + r < k_end && base + r >= k_lo && page_ok[k] && col_ok;
             cp_async16(smem_u32(dst) + tile_off<DIM>(r, c), srcs[k], ok);
         }
     };
@@ -146,8 +153,8 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
         const bool first = tile < kept_tiles;
         const int base = first ? tile * kTileKeys : k_begin + (tile - kept_tiles) * kTileKeys;
         const int from = first ? 0 : k_lo, to = first ? kept : k_end;       // the keys of this tile that are read
-        load_rows(std::integral_constant<int, D>{}, kbase, base, head_off, from, to);
-        load_rows(std::integral_constant<int, DV>{}, kbase + kTileBytes, base, v_off, from, to);
+        load_rows(std::integral_constant<int, D>{}, d_real, kbase, base, head_off, from, to);
+        load_rows(std::integral_constant<int, DV>{}, dv_real, kbase + kTileBytes, base, v_off, from, to);
     };
 
     for (int s = 0; s < kStages - 1; ++s) {
@@ -261,12 +268,17 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
         // the sink's term 2^(0 - m): it grows beyond the type only where the keys hold nothing (the output is 0 then)
         if (opt.sink) l_run[h] += exp2f(sink_log2(opt, head[h]) - m_run[h] * scale_log2);
         const float inv = 1.f / l_run[h];
-        __nv_bfloat16* dst = out + ((size_t)tok[h] * hq + head[h]) * DV;
-        const __nv_bfloat16* gp = opt.gate != nullptr ? opt.gate + (size_t)tok[h] * opt.gate_pitch + (size_t)head[h] * DV : nullptr;
+        __nv_bfloat16* dst = out + ((size_t)tok[h] * hq + head[h]) * dv_real;
+        const __nv_bfloat16* gp = opt.gate != nullptr ? gate_of(opt, tok[h], head[h], dv_real) : nullptr;
+        const float head_gate = gp != nullptr && opt.gate_per_head ? __bfloat162float(*gp) : 0.f;
 #pragma unroll
         for (int i = 0; i < DV / 8; ++i) {
+            if (PAD && i * 8 >= dv_real) break;
             float a = o[i][2 * h] * inv, b = o[i][2 * h + 1] * inv;
-            if (gp != nullptr) {
+            if (gp != nullptr && opt.gate_per_head) {
+                a = gated_by(a, head_gate);
+                b = gated_by(b, head_gate);
+            } else if (gp != nullptr) {
                 if (gate_vec) {       // the thread's two neighbours in one load
                     const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp + i * 8 + 2 * t4));
                     a = gated_by(a, g.x);
@@ -281,15 +293,15 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     }
 }
 
-template <int D, int DV>
+template <int D, int DV, bool PAD>
 static int launch(const void* q, const void* cache, const int* table, int table_stride, const int* seq_rows,
                   const int* cu_q, const int* kv_len, void* out, int entries, int max_q_len, int hq, int hkv,
-                  int page_size, float scale, int window, int num_pages, int* error, const SoftmaxOptions& opt,
+                  int page_size, float scale, int window, int num_pages, int* error, const SoftmaxOptions& opt, int d, int dv,
                   cudaStream_t stream) {
     const size_t smem = (size_t)kStages * kTileKeys * (D + DV) * 2;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<D, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<D, DV, PAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
@@ -297,9 +309,9 @@ static int launch(const void* q, const void* cache, const int* table, int table_
     const int row_tiles = ceil_div(max_q_len * group, kTileRows);
     if (row_tiles > 65535) return SE_ERR_UNSUPPORTED;
     dim3 grid(hkv, row_tiles, entries);
-    attn_prefill_kernel<D, DV><<<grid, kThreads, smem, stream>>>(
+    attn_prefill_kernel<D, DV, PAD><<<grid, kThreads, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, table, table_stride, seq_rows, cu_q, kv_len,
-        (__nv_bfloat16*)out, hq, hkv, page_size, scale * 1.4426950408889634f, window, num_pages, error, opt);
+        (__nv_bfloat16*)out, hq, hkv, page_size, scale * 1.4426950408889634f, window, num_pages, error, opt, d, dv);
     return (int)cudaGetLastError();
 }
 
@@ -314,21 +326,29 @@ extern "C" int se_attn_prefill(const void* q, const void* cache, const int* tabl
                                int max_q_len, int hq, int hkv, int head_dim, int v_head_dim, int page_size, float scale,
                                int window, int num_pages, int* error, float softcap, int sink, const void* gate,
                                int gate_pitch, const float* sink_logits, int keep_first, const float* slopes,
-                               cudaStream_t stream) {
+                               int gate_per_head, cudaStream_t stream) {
     if (entries <= 0 || max_q_len <= 0) return 0;
-    if (!(head_dim == 64 || head_dim == 128) || hkv <= 0 || hq % hkv || entries > 65535 || hkv > 65535)
+    if (head_dim <= 0 || head_dim > 128 || head_dim % 8 || v_head_dim <= 0 || v_head_dim > 128 || v_head_dim % 8 || hkv <= 0 || hq % hkv || entries > 65535 || hkv > 65535)
         return SE_ERR_UNSUPPORTED;
-    if (softcap < 0.f || !(scale > 0.f) || (gate != nullptr && gate_pitch < hq * v_head_dim) || keep_first < 0)
+    if (softcap < 0.f || !(scale > 0.f) || (gate != nullptr && gate_pitch < (gate_per_head ? hq : hq * v_head_dim)) || keep_first < 0)
         return SE_ERR_ARGUMENT;
     const se::mma::SoftmaxOptions opt{softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f,
                                       sink || sink_logits != nullptr, (const __nv_bfloat16*)gate, gate_pitch, sink_logits,
-                                      window > 0 ? keep_first : 0, slopes, 1.f / scale};
+                                      window > 0 ? keep_first : 0, slopes, 1.f / scale, gate_per_head};
+    // tiles of 64 or 128 query/key columns and 32, 64 or 128 value columns; head sizes between them in the next wider tile
+    const int dt = head_dim <= 64 ? 64 : 128, dvt = v_head_dim <= 32 ? 32 : v_head_dim <= 64 ? 64 : 128;
+    const bool pad = dt != head_dim || dvt != v_head_dim;
+#define SE_PREFILL_LAUNCH(DQ, DVAL, PAD)                                                                               \
+    return se::pre::launch<DQ, DVAL, PAD>(q, cache, table, table_stride, seq_rows, cu_q, kv_len, out, entries, max_q_len, \
+                                          hq, hkv, page_size, scale, window, num_pages, error, opt, head_dim, v_head_dim, stream)
 #define SE_PREFILL_CASE(DQ, DVAL)                                                                                      \
-    if (head_dim == DQ && v_head_dim == DVAL)                                                                          \
-        return se::pre::launch<DQ, DVAL>(q, cache, table, table_stride, seq_rows, cu_q, kv_len, out, entries, max_q_len, \
-                                         hq, hkv, page_size, scale, window, num_pages, error, opt, stream);
+    if (dt == DQ && dvt == DVAL) {                                                                                     \
+        if (pad) SE_PREFILL_LAUNCH(DQ, DVAL, true);                                                                    \
+        SE_PREFILL_LAUNCH(DQ, DVAL, false);                                                                            \
+    }
     SE_PREFILL_CASE(64, 64) SE_PREFILL_CASE(128, 128) SE_PREFILL_CASE(64, 32) SE_PREFILL_CASE(64, 128)
     SE_PREFILL_CASE(128, 64) SE_PREFILL_CASE(128, 32)
+#undef SE_PREFILL_LAUNCH
 #undef SE_PREFILL_CASE
     return SE_ERR_UNSUPPORTED;
 }

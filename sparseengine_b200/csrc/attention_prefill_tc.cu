@@ -173,7 +173,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
     const int last_row = min(row_base + kTiles * kRows, total_rows) - 1;
     const int max_pos = q_start + last_row / group;
     const int first_pos = q_start + row_base / group;
-    const int k_lo = window > 0 ? max(0, first_pos - window + 1) : 0;
+    const int k_lo = first_visible(first_pos, window);
     const int k_begin = (k_lo / kKeys) * kKeys;
     const int k_end = max_pos + 1;
     // first keys that stay visible beside a window: those before the CTA's window come as tiles of their own, ahead
@@ -328,7 +328,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         const bool valid = row < total_rows;
         const int rr = valid ? row : total_rows - 1;
         const int pos = q_start + rr / group;
-        const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+        const int lo = first_visible(pos, window);
         const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
         float m_ref = -INFINITY, l = 0.f;                  // reference maximum (log2 units), running sum
         const float slope = se::mma::raw_slope(opt, kvh * group + rr % group);      // distance bias per token, raw units
@@ -443,9 +443,11 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             if (opt.sink) l += exp2f(se::mma::sink_log2(opt, kvh * group + rr % group) - m_ref);
             const float inv = 1.f / l;
             __nv_bfloat16* dst = out + ((size_t)(tok0 + rr / group) * hq + kvh * group + rr % group) * D;
-            const bool gate_vec = opt.gate != nullptr && se::mma::gate_rows_aligned(opt, 16);
+            const bool gate_vec = opt.gate != nullptr && !opt.gate_per_head && se::mma::gate_rows_aligned(opt, 16);
             const __nv_bfloat16* gp = opt.gate != nullptr
-                ? opt.gate + (size_t)(tok0 + rr / group) * opt.gate_pitch + (size_t)(kvh * group + rr % group) * D : nullptr;
+                ? se::mma::gate_of(opt, tok0 + rr / group, kvh * group + rr % group, D) : nullptr;
+            const float inv_gated = gp != nullptr && opt.gate_per_head ? se::mma::gated(inv, gp) : inv;     // one gate per head: in the factor
+            const bool gate_each = gp != nullptr && !opt.gate_per_head;
 #pragma unroll 1
             for (int c0 = 0; c0 < D; c0 += 32) {
                 uint32_t ov[32];
@@ -456,12 +458,12 @@ attn_prefill_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                     for (int c = 0; c < 32; c += 8) {
                         uint32_t w[4];
                         uint4 graw = make_uint4(0u, 0u, 0u, 0u);           // eight gate values in one load where the rows allow it
-                        if (gp != nullptr && gate_vec) graw = *reinterpret_cast<const uint4*>(gp + c0 + c);
+                        if (gate_each && gate_vec) graw = *reinterpret_cast<const uint4*>(gp + c0 + c);
                         const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&graw);
 #pragma unroll
                         for (int i = 0; i < 4; ++i) {
-                            float a = __uint_as_float(ov[c + 2 * i]) * inv, b = __uint_as_float(ov[c + 2 * i + 1]) * inv;
-                            if (gp != nullptr) {
+                            float a = __uint_as_float(ov[c + 2 * i]) * inv_gated, b = __uint_as_float(ov[c + 2 * i + 1]) * inv_gated;
+                            if (gate_each) {
                                 if (gate_vec) {
                                     const float2 g = __bfloat1622float2(g2[i]);
                                     a = se::mma::gated_by(a, g.x);
@@ -501,15 +503,15 @@ extern "C" int se_attn_prefill_tc(const void* q, const void* cache, const int* t
                                   const int* seq_rows, const int* cu_q, const int* kv_len, void* out, int* error,
                                   int entries, int max_q_len, int hq, int hkv, int head_dim, int page_size, float scale,
                                   int window, int num_pages, float softcap, int sink, const void* gate, int gate_pitch,
-                                  const float* sink_logits, int keep_first, const float* slopes, cudaStream_t stream) {
+                                  const float* sink_logits, int keep_first, const float* slopes, int gate_per_head, cudaStream_t stream) {
     using namespace se::fa;
     if (entries <= 0 || max_q_len <= 0) return 0;
     if (!se_attn_prefill_tc_supported(head_dim, hq, hkv) || entries > 65535 || hkv > 65535) return SE_ERR_UNSUPPORTED;
-    if (softcap < 0.f || !(scale > 0.f) || (gate != nullptr && gate_pitch < hq * head_dim) || keep_first < 0)
+    if (softcap < 0.f || !(scale > 0.f) || (gate != nullptr && gate_pitch < (gate_per_head ? hq : hq * head_dim)) || keep_first < 0)
         return SE_ERR_ARGUMENT;
     const se::mma::SoftmaxOptions opt{softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f,
                                       sink || sink_logits != nullptr, (const __nv_bfloat16*)gate, gate_pitch, sink_logits,
-                                      window > 0 ? keep_first : 0, slopes, 1.f / scale};
+                                      window > 0 ? keep_first : 0, slopes, 1.f / scale, gate_per_head};
     const size_t smem = (size_t)kTiles * kQBytes + kStages * kKVStageBytes + 1024;
     static bool configured = false;
     if (!configured) {

@@ -109,6 +109,14 @@ inline cudaError_t launch_dependent_if(bool dependent, void (*kernel)(KArgs...),
 #define SE_LAUNCH_DEPENDENT_IF(cond, tag, ...) \
     ([&] { static const bool on = se::pdl_enabled(tag); return se::launch_dependent_if(on && (cond), __VA_ARGS__); }())
 
+// The first key a query at `pos` sees.  window > 0: the last `window` keys up to its own; window < 0: the keys of
+// its own chunk, chunks of -window positions counted from position 0; window = 0: every key.  It never falls as
+// `pos` grows, so the first row of a tile of rows gives the first key the tile needs.
+__host__ __device__ __forceinline__ int first_visible(int pos, int window) {
+    if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
+    return window < 0 ? pos - pos % -window : 0;
+}
+
 // Codes a kernel writes into the library's error word (one int per device, 0 = fine; the
 // first failure stays).  1..19: a bounded wait on a barrier ran out (the number names the
 // waiting role).  From 20: an index a kernel was given points outside what it may touch; the

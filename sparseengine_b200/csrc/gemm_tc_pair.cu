@@ -490,7 +490,7 @@ extern "C" int se_moe_grouped_gemm_pair(int mode, const void* a, const void* w, 
                                         int max_tiles, int n_out, int k_dim, int act_kind, float act_limit,
                                         float act_alpha, cudaStream_t stream) {
     if (assignments <= 0 || max_tiles <= 0) return 0;
-    if (act_kind != SE_GLU_SILU && act_kind != SE_GLU_CLAMPED) return SE_ERR_ARGUMENT;
+    if (act_kind < SE_GLU_SILU || act_kind > SE_GLU_GELU) return SE_ERR_ARGUMENT;
     if (!se_moe_grouped_gemm_pair_supported(k_dim, n_out) || (mode != 0 && mode != 1)) return SE_ERR_UNSUPPORTED;
     const int w_rows = mode == 0 ? 2 * n_out : n_out;
     CUtensorMap mw, mx;

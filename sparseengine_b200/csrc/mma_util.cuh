@@ -49,7 +49,8 @@ template <int D> __device__ __forceinline__ uint32_t tile_off(int r, int c) {
 //                     capped score goes back to raw units: s <- cap_out * tanh(s * cap_in).
 //   sink            : a key of score 0 without a value joins the softmax's denominator.
 //   gate, gate_pitch: the output is multiplied element by element with sigmoid(gate[t][h * dv + i])
-//                     (rows gate_pitch elements apart); nullptr: no gate.
+//                     (rows gate_pitch elements apart); nullptr: no gate.  gate_per_head: one number per head,
+//                     sigmoid(gate[t][h]).
 //   sink_logits     : with `sink`, a learned logit per query head in the place of the sink's 0 (unscaled); nullptr: 0.
 //   keep_first      : with a window, keys 0 .. keep_first-1 stay visible beside the window's.
 //   slopes          : a distance bias: the scaled score of query position i and key position j becomes
@@ -64,6 +65,7 @@ struct SoftmaxOptions {
     int keep_first;
     const float* slopes;
     float inv_scale;
+    int gate_per_head;
 };
 // what a head's raw scores lose per token of distance
 __device__ __forceinline__ float raw_slope(const SoftmaxOptions& opt, int head) {
@@ -152,6 +154,10 @@ __device__ __forceinline__ float gated_by(float o, float g) {
 }
 __device__ __forceinline__ float gated(float o, const __nv_bfloat16* gate) {
     return gated_by(o, __bfloat162float(*gate));
+}
+// Where the gate of element 0 of a head's output lies; with one gate per head it is the head's only one.
+__device__ __forceinline__ const __nv_bfloat16* gate_of(const SoftmaxOptions& opt, size_t token, size_t head, int dv) {
+    return opt.gate + token * opt.gate_pitch + (opt.gate_per_head ? head : head * dv);
 }
 // Whether the gate's rows can be read 16 bytes (8 elements) or 4 bytes (2 elements) at a time, for head
 // sizes that are multiples of 8.

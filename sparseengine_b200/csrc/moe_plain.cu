@@ -408,7 +408,7 @@ extern "C" int se_moe_grouped_gemm_plain(int mode, const void* a, const void* w,
                                          int top_k, int act_kind, float act_limit, float act_alpha, int dtype,
                                          cudaStream_t stream) {
     if (max_tiles <= 0) return 0;
-    if (act_kind != SE_GLU_SILU && act_kind != SE_GLU_CLAMPED) return SE_ERR_ARGUMENT;
+    if (act_kind < SE_GLU_SILU || act_kind > SE_GLU_GELU) return SE_ERR_ARGUMENT;
     dim3 grid(max_tiles, se::ceil_div(n_out, se::kBN));
     SE_DISPATCH_DTYPE(dtype, T, {
         if (mode == 0)

@@ -46,6 +46,7 @@ LIMITS = {
     "router_max_unaligned_width": 6400,     # widths that are no multiple of 4 keep 8 token rows in shared memory
     "moe_max_experts": 6079,                # the routing build's scans keep two ints per expert in shared memory
     "attention_max_head_dim": 256,          # in steps of 16
+    "sandwich_norm_max_width": 51200,       # as the RMS norm: a row that is not kept in registers lies in shared memory
     "layernorm_max_width": 51200,           # as the RMS norm: the row is kept in shared memory in 32-bit
     "recurrent_max_state_rows": 512,        # rows of a recurrence's state on the key/state side (16 registers x 32 lanes)
     "latent_max_row": 1024,                 # latent plus shared key part of one position (32 registers x 32 lanes)
@@ -210,6 +211,25 @@ def _sink_logits(sink, num_heads: int):
     return _ptr(sink, torch.float32, "sink")
 
 
+def _visible_arg(window, chunk) -> int:
+    """The attention kernels' one argument for what a query sees: n > 0 a window, -n a chunk, 0 every key."""
+    if window and chunk:
+        raise ValueError("attention has a window or a chunk, not both")
+    if (window is not None and window < 0) or (chunk is not None and chunk < 0):
+        raise ValueError("a window or a chunk has a positive size")
+    return -int(chunk) if chunk else int(window or 0)
+
+
+def _gate_per_head(gate, num_heads: int, v_head_dim: int) -> int:
+    """1 if the gate's matrix has one column per head, 0 if one per output element (or there is no gate)."""
+    if gate is None:
+        return 0
+    if gate.shape[1] not in (num_heads, num_heads * v_head_dim):
+        raise ValueError(f"gate must have {num_heads} columns (one per head) or {num_heads * v_head_dim} (one per output element), "
+                         f"got {gate.shape[1]}")
+    return int(gate.shape[1] == num_heads and v_head_dim != 1)
+
+
 def _slopes_ptr(slopes, num_heads: int):
     if slopes is not None and slopes.shape != (num_heads,):
         raise ValueError(f"a distance bias has one slope per query head ({num_heads}), got {tuple(slopes.shape)}")
@@ -218,12 +238,13 @@ def _slopes_ptr(slopes, num_heads: int):
 
 def paged_attention_plain(q, cache, table, seq_rows, token_seq, positions, out, *, num_heads, num_kv_heads,
                           head_dim, page_size, scale, window=None, num_pages=None, v_head_dim=None, softcap=None,
-                          sink=False, gate=None, keep_first: int = 0, slopes=None):
+                          sink=False, gate=None, keep_first: int = 0, slopes=None, chunk=None):
     """``v_head_dim``: the values' head size where it differs from the queries' and keys'.
     ``softcap`` c: scaled scores become c tanh(s / c).  ``sink``: True: a key of score 0 without a value
     joins the softmax's denominator; a 32-bit tensor [num_heads]: its logit is the head's entry (unscaled).
     ``gate``: a matrix (rows may be a view with a pitch) whose sigmoid multiplies the output,
-    [tokens, num_heads * v_head_dim].  ``keep_first`` n (with a window): keys 0..n-1 stay visible.
+    [tokens, num_heads * v_head_dim], or [tokens, num_heads]: one number per head.  ``chunk`` n (instead of a
+    window): a query sees the keys of its own run of n positions, counted from position 0.  ``keep_first`` n (with a window): keys 0..n-1 stay visible.
     ``slopes`` (32-bit, [num_heads]): the score of query position i and key position j loses
     ``slopes[head] * (i - j)``."""
     tokens = q.shape[0]
@@ -231,15 +252,16 @@ def paged_attention_plain(q, cache, table, seq_rows, token_seq, positions, out, 
     if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1 or gate.dtype != dt):
         raise ValueError("gate must be a matrix of q's dtype with contiguous rows")
     sink_logits = _sink_logits(sink, num_heads)
-    _check(_fn("se_paged_attention_plain", "pppipppp" "iiiiii" "f" "iip" "fipi" "pip" "ip")(
+    per_head = _gate_per_head(gate, num_heads, int(v_head_dim or head_dim))
+    _check(_fn("se_paged_attention_plain", "pppipppp" "iiiiii" "f" "iip" "fipi" "pip" "iip")(
         _ptr(q, None, "q"), _ptr(cache, dt, "cache"), _ptr(table, torch.int32, "table"), table.shape[1],
         _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(token_seq, torch.int32, "token_seq"),
         _ptr(positions, torch.int32, "positions"), _ptr(out, dt, "out"), tokens, num_heads, num_kv_heads,
-        head_dim, int(v_head_dim or head_dim), page_size, float(scale), int(window or 0),
+        head_dim, int(v_head_dim or head_dim), page_size, float(scale), _visible_arg(window, chunk),
         cache.shape[0] if num_pages is None else int(num_pages), _ptr(error_word(q.device)),
         float(softcap or 0.0), _has_sink(sink), gate.data_ptr() if gate is not None else None,
         gate.stride(0) if gate is not None else 0, sink_logits, int(keep_first or 0), _slopes_ptr(slopes, num_heads),
-        dtype_code(dt), _stream()),
+        per_head, dtype_code(dt), _stream()),
         "paged_attention_plain")
     return out
 
@@ -247,7 +269,7 @@ def paged_attention_plain(q, cache, table, seq_rows, token_seq, positions, out, 
 def qk_prep_general(proj, q_w, k_w, positions, token_seq, seq_rows, table, cache, q_out, *, num_heads, num_kv_heads,
                     head_dim, v_head_dim, eps, page_size, has_kv=True, temperature=None, num_pages=None,
                     inv_freq=None, rotary_dim: int = 0, v_first=None, v_mix=None, bias=None, per_head: bool = False,
-                    per_head_unit: bool = False):
+                    per_head_unit: bool = False, pairing: str = "split_half", rope_scale: float = 1.0):
     """Query/key preparation in 32-bit, rounded once: whole-projection RMS norms (optional), a rotation
     of the first ``rotary_dim`` dims of every head (split halves, angles ``position * inv_freq``), a query
     temperature ``(coef, every)`` (q times 1 + coef ln(floor((p+1)/every) + 1)), keys and values of
@@ -256,7 +278,10 @@ def qk_prep_general(proj, q_w, k_w, positions, token_seq, seq_rows, table, cache
     number on the device): the values written are ``(1 - v_mix) v + v_mix v_first``.
     ``bias`` (32-bit, one per column of the projection row): added before anything else.  ``per_head``: the
     norms are per head, with weights of ``head_dim`` elements shared by the heads; ``per_head_unit``: per head
-    without weights."""
+    without weights, over the rotated head.  ``pairing``: "split_half" or "interleaved" (neighbours rotate into one
+    another); ``rope_scale`` multiplies cos and sin."""
+    if pairing not in ("split_half", "interleaved"):
+        raise ValueError(f"qk_prep_general: pairing {pairing!r} is not 'split_half' or 'interleaved'")
     tokens = proj.shape[0]
     if per_head_unit and (per_head or q_w is not None or k_w is not None):
         raise ValueError("qk_prep_general: per_head_unit is a norm without weights")
@@ -268,7 +293,7 @@ def qk_prep_general(proj, q_w, k_w, positions, token_seq, seq_rows, table, cache
     coef, every = (float(temperature[0]), int(temperature[1])) if temperature else (0.0, 0)
     if v_first is not None and (v_first.dim() != 2 or v_first.stride(1) != 1 or v_first.dtype != dt or v_mix is None):
         raise ValueError("v_first must be a matrix of proj's dtype with contiguous rows, and comes with v_mix")
-    _check(_fn("se_qk_prep_general", "pipp" "pipip" "ppp" "pi" "pp" "iiiii" "f" "fi" "iiip" "pi" "ip")(
+    _check(_fn("se_qk_prep_general", "pipp" "pipip" "ppp" "pi" "pp" "iiiii" "f" "fi" "iiip" "pi" "if" "ip")(
         proj.data_ptr(), proj.stride(0), _ptr(q_w, dt, "q_norm"), _ptr(k_w, dt, "k_norm"),
         _ptr(inv_freq, torch.float32, "inv_freq"), int(rotary_dim), v_first.data_ptr() if v_first is not None else None,
         v_first.stride(0) if v_first is not None else 0, _ptr(v_mix, torch.float32, "v_mix") if v_first is not None else None,
@@ -277,7 +302,8 @@ def qk_prep_general(proj, q_w, k_w, positions, token_seq, seq_rows, table, cache
         _ptr(cache, dt, "cache") if has_kv else None, _ptr(q_out, dt, "q_out"), tokens, num_heads, num_kv_heads, head_dim,
         int(v_head_dim), float(eps), coef, every, page_size, int(bool(has_kv)),
         (cache.shape[0] if num_pages is None else int(num_pages)) if has_kv else 0, _ptr(error_word(proj.device)),
-        _ptr(bias, torch.float32, "bias"), 2 if per_head_unit else int(bool(per_head)), dtype_code(dt), _stream()), "qk_prep_general")
+        _ptr(bias, torch.float32, "bias"), 2 if per_head_unit else int(bool(per_head)), int(pairing == "interleaved"),
+        float(rope_scale), dtype_code(dt), _stream()), "qk_prep_general")
     return q_out
 
 
@@ -346,6 +372,41 @@ def add_rmsnorm_stream(x, y, w, eps: float, out32=None, out_act=None, alpha: flo
         _ptr(out_act, dt, "out_act"), rows, hidden, float(eps), int(groups), _ptr(table, dt, "inject table"),
         _ptr(ids, torch.int32, "inject ids"), table.shape[0] if table is not None else 0, float(scale),
         _ptr(step, torch.float32, "inject step"), dtype_code(dt), _stream()), "add_rmsnorm_stream")
+
+
+def sandwich_norm(stream, y, *, post=None, following=None, out=None, rows=None, store: bool = True, dtype=None):
+    """Between two sublayers of a model that norms before and after each (csrc/sandwich_norm.cu), per row and in 32-bit:
+    ``c = y``; ``y`` may be ``((y0, w0, s0), (y1, w1, s1), eps)``: two results side by side, ``c = s0 rms(y0) w0 + s1 rms(y1)
+    w1``; ``post = (w, eps)``: ``c <- rms(c) w``; ``x = stream + c`` (``stream`` may be None), stored back with ``store``;
+    ``out`` receives ``rms(x) w`` with ``following = (w, eps)``, else ``x``, in its own type.  ``y`` None: ``x = stream``.
+    ``rows`` (int32, on the device; without ``store``): the stream's and results' row of every row of ``out``."""
+    y0 = y1 = w0 = w1 = None
+    s0 = s1 = eps_pair = 0.0
+    if isinstance(y, tuple):
+        (y0, w0, s0), (y1, w1, s1), eps_pair = y
+    else:
+        y0 = y
+    some = next(t for t in (y0, stream) if t is not None)
+    rows_in, hidden = some.shape
+    dt = dtype or (out.dtype if out is not None else y0.dtype if y0 is not None else torch.float32)
+    n = rows.numel() if rows is not None else rows_in
+    for t in (y0, y1, stream):
+        if t is not None and tuple(t.shape) != (rows_in, hidden):
+            raise ValueError("sandwich_norm: the stream and the results must have one shape")
+    for w in (w0, w1, post and post[0], following and following[0]):
+        if w is not None and w.shape != (hidden,):
+            raise ValueError(f"norm weight shape {tuple(w.shape)} does not match width {hidden}")
+    if out is not None and tuple(out.shape) != (n, hidden):
+        raise ValueError("sandwich_norm: out must have a row per row asked for")
+    post_w, post_eps = post if post is not None else (None, 0.0)
+    next_w, next_eps = following if following is not None else (None, 0.0)
+    store = bool(store) and stream is not None
+    _check(_fn("se_sandwich_norm", "ppppp" "fff" "pfpf" "pp" "iiii" "ip")(
+        _ptr(stream, torch.float32, "stream"), _ptr(y0, dt, "y"), _ptr(y1, dt, "y"), _ptr(w0, dt, "w"), _ptr(w1, dt, "w"),
+        float(s0), float(s1), float(eps_pair), _ptr(post_w, dt, "post weight"), float(post_eps), _ptr(next_w, dt, "norm weight"),
+        float(next_eps), _ptr(out, dt, "out"), _ptr(rows, torch.int32, "rows"), rows_in, n, hidden, int(store), dtype_code(dt),
+        _stream()), "sandwich_norm")
+    return out
 
 
 def sigmoid_gate_(x, gate):
@@ -496,20 +557,28 @@ def latent_attention_tiled(qfull, cache, table, seq_rows, cu_q, kv_len, sink, ou
 
 # ---- retention (csrc/retention.cu) ----------------------------------------------------------------
 
-def retention_prep(proj, q_off: int, k_off: int, inv_freq, positions, q32, k32, *, heads, head_dim, rotary_dim, k_scale):
+def retention_prep(proj, q_off: int, k_off: int, inv_freq, positions, q32, k32, *, heads, head_dim, rotary_dim, k_scale,
+                   silu: bool = False):
+    """q32 and k32 in 32-bit: rotated, k times ``k_scale``; with ``silu`` the activation comes first."""
     tokens = proj.shape[0]
-    _check(_fn("se_retention_prep", "piii" "pp" "pp" "iiii" "f" "ip")(
+    _check(_fn("se_retention_prep", "piii" "pp" "pp" "iiii" "fi" "ip")(
         proj.data_ptr(), proj.stride(0), int(q_off), int(k_off), _ptr(inv_freq, torch.float32, "inv_freq"),
         _ptr(positions, torch.int32, "positions"), _ptr(q32, torch.float32, "q32"), _ptr(k32, torch.float32, "k32"),
-        tokens, heads, head_dim, rotary_dim, float(k_scale), dtype_code(proj.dtype), _stream()), "retention_prep")
+        tokens, heads, head_dim, rotary_dim, float(k_scale), int(silu), dtype_code(proj.dtype), _stream()), "retention_prep")
 
 
-def retention_scan(q32, k32, proj, v_off: int, decay, state, step, o, *, heads, head_dim, v_head_dim):
-    _check(_fn("se_retention_scan", "pp" "pii" "p" "pl" "pp" "p" "iiii" "ip")(
+def retention_scan(q32, k32, proj, v_off: int, decay, state, step, o, *, heads, head_dim, v_head_dim, silu: bool = False,
+                   qk=None):
+    """``silu``: the values are silu of the projection's columns.  ``qk`` (with ``q32`` and ``k32`` None): ``(q_off,
+    k_off, k_scale)``, q and k straight from the projection's columns (silu too), without a rotation."""
+    if (qk is None) != (q32 is not None) or (q32 is None) != (k32 is None):
+        raise ValueError("retention_scan takes q32 and k32, or qk")
+    q_off, k_off, k_scale = qk if qk is not None else (0, 0, 1.0)
+    _check(_fn("se_retention_scan", "pp" "pii" "p" "pl" "pp" "p" "iiii" "iiif" "ip")(
         _ptr(q32, torch.float32, "q32"), _ptr(k32, torch.float32, "k32"), proj.data_ptr(), proj.stride(0), int(v_off),
         _ptr(decay, torch.float32, "decay"), _ptr(state, torch.float32, "state"), state.stride(0), _ptr(step.cu_q),
         _ptr(step.seq_rows), _ptr(o, torch.float32, "o"), step.num_seqs, heads, head_dim, v_head_dim,
-        dtype_code(proj.dtype), _stream()), "retention_scan")
+        int(silu), int(q_off), int(k_off), float(k_scale), dtype_code(proj.dtype), _stream()), "retention_scan")
     return o
 
 
@@ -532,7 +601,8 @@ def retention_segment_plan(entries: int, heads: int, v_head_dim: int, max_q_len:
     return (segs, seg_len) if segs > 1 else (1, 0)
 
 
-def retention_chunk(q32, k32, proj, v_off: int, decay, state, step, o, *, heads, head_dim, v_head_dim, segments=None):
+def retention_chunk(q32, k32, proj, v_off: int, decay, state, step, o, *, heads, head_dim, v_head_dim, segments=None,
+                    silu: bool = False):
     """The same recurrence as :func:`retention_scan` in chunks of 64 tokens (closed form per chunk, 32-bit
     FMA arithmetic): for steps that bring prompt portions.  ``segments``: ``(per entry, tokens each)``, default
     by :func:`retention_segment_plan`."""
@@ -543,11 +613,11 @@ def retention_chunk(q32, k32, proj, v_off: int, decay, state, step, o, *, heads,
     if max_seg > 1:
         seg_state = torch.empty(step.num_seqs * max_seg * heads * head_dim * v_head_dim, dtype=torch.float32, device=q32.device)
         launch_count += 2
-    _check(_fn("se_retention_chunk", "pp" "pii" "p" "pl" "pp" "p" "iiii" "iip" "ip")(
+    _check(_fn("se_retention_chunk", "pp" "pii" "p" "pl" "pp" "p" "iiii" "iipi" "ip")(
         _ptr(q32, torch.float32, "q32"), _ptr(k32, torch.float32, "k32"), proj.data_ptr(), proj.stride(0), int(v_off),
         _ptr(decay, torch.float32, "decay"), _ptr(state, torch.float32, "state"), state.stride(0), _ptr(step.cu_q),
         _ptr(step.seq_rows), _ptr(o, torch.float32, "o"), step.num_seqs, heads, head_dim, v_head_dim, int(max_seg),
-        int(seg_len), _ptr(seg_state), dtype_code(proj.dtype), _stream()), "retention_chunk")
+        int(seg_len), _ptr(seg_state), int(silu), dtype_code(proj.dtype), _stream()), "retention_chunk")
     return o
 
 
@@ -556,6 +626,18 @@ def retention_out(o, proj, g_off: int, out, *, heads, v_head_dim, eps):
     _check(_fn("se_retention_out", "ppii" "p" "iii" "f" "ip")(
         _ptr(o, torch.float32, "o"), proj.data_ptr(), proj.stride(0), int(g_off), _ptr(out, proj.dtype, "out"), tokens,
         heads, v_head_dim, float(eps), dtype_code(proj.dtype), _stream()), "retention_out")
+    return out
+
+
+def retention_out_joint(o, proj, g_off: int, w, out, *, eps):
+    """out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) over the concatenated heads (a row of ``out``); the gate is
+    the projection's columns from ``g_off`` on."""
+    tokens, width = out.shape
+    if w.shape != (width,):
+        raise ValueError(f"the norm's weight has {tuple(w.shape)} elements, the concatenated heads {width}")
+    _check(_fn("se_retention_out_joint", "ppii" "pp" "ii" "f" "ip")(
+        _ptr(o, torch.float32, "o"), _rows_ptr(proj, "proj"), proj.stride(0), int(g_off), _ptr(w, proj.dtype, "w"),
+        _ptr(out, proj.dtype, "out"), tokens, width, float(eps), dtype_code(proj.dtype), _stream()), "retention_out_joint")
     return out
 
 
@@ -870,8 +952,9 @@ def moe_max_tiles(assignments: int, experts: int, tile_rows: int) -> int:
 
 
 # Gated activations of the experts' first product: ``silu`` is silu(gate) * up; ``clamped_swiglu`` is
-# g sigmoid(alpha g) (u + 1) with g = min(gate, limit) and u = clamp(up, -limit, limit).
-GLU_KINDS = {"silu": 0, "clamped_swiglu": 1}
+# g sigmoid(alpha g) (u + 1) with g = min(gate, limit) and u = clamp(up, -limit, limit); ``gelu_tanh`` is gelu(gate) * up
+# with gelu in its tanh form.
+GLU_KINDS = {"silu": 0, "clamped_swiglu": 1, "gelu_tanh": 2}
 
 
 def _glu_args(activation):
@@ -1059,7 +1142,7 @@ def gemm_tc_dense(x, w, out, nt: int = 128):
 def attn_decode_supported(head_dim: int, num_heads: int, num_kv_heads: int) -> bool:
     """What ``se_attn_decode_supported`` of the library answers, restated here so that asking does not
     compile the kernel for a model that cannot use it (a GPU test compares the two)."""
-    return head_dim in (64, 128) and num_kv_heads > 0 and num_heads % num_kv_heads == 0
+    return 0 < head_dim <= 128 and head_dim % 8 == 0 and num_kv_heads > 0 and num_heads % num_kv_heads == 0
 
 
 _sm_counts: dict = {}
@@ -1101,28 +1184,28 @@ def attn_decode_plan(tokens: int, num_heads: int, num_kv_heads: int, max_keys: i
 
 def _softmax_options(q, gate, num_heads, v_head_dim, softcap, sink, keep_first, slopes):
     """The tail of the tensor-core attention kernels' arguments: cap, sink, gate pointer, gate pitch, the learned
-    sink's logits, the count of first keys that stay visible, and the distance bias's slopes."""
-    if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1 or gate.dtype != q.dtype
-                             or gate.shape[1] != num_heads * v_head_dim):
-        raise ValueError("gate must be a matrix [tokens, heads * value size] of q's dtype with contiguous rows")
+    sink's logits, the count of first keys that stay visible, the distance bias's slopes, and whether the gate has one
+    number per head."""
+    if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1 or gate.dtype != q.dtype):
+        raise ValueError("gate must be a matrix of q's dtype with contiguous rows")
     return (float(softcap or 0.0), _has_sink(sink), gate.data_ptr() if gate is not None else None,
             gate.stride(0) if gate is not None else 0, _sink_logits(sink, num_heads), int(keep_first),
-            _slopes_ptr(slopes, num_heads))
+            _slopes_ptr(slopes, num_heads), _gate_per_head(gate, num_heads, v_head_dim))
 
 
 def attn_decode_value_dim_supported(v_head_dim: int) -> bool:
     """Value head sizes the tensor-core kernels take beside a query/key head size they take."""
-    return v_head_dim in (32, 64, 128)
+    return 0 < v_head_dim <= 128 and v_head_dim % 8 == 0
 
 
 def attn_decode(q, cache, table, seq_rows, token_seq, positions, out, *, num_heads, num_kv_heads, head_dim, page_size,
                 scale, window=None, max_keys: int, num_pages=None, step_inputs_settled: bool = False, v_head_dim=None,
-                softcap=None, sink=False, gate=None, keep_first: int = 0, slopes=None):
+                softcap=None, sink=False, gate=None, keep_first: int = 0, slopes=None, chunk=None):
     """``step_inputs_settled``: ``table``, ``seq_rows``, ``token_seq`` and ``positions`` were complete
     before the kernel launched just before this call began (that kernel wrote ``q`` and the step's
     keys).  The attention kernel, launched as its dependent, then finds its place in the block table
     while it still runs; otherwise it waits for it first.  ``v_head_dim``, ``softcap``, ``sink``,
-    ``gate`` and ``slopes`` as :func:`paged_attention_plain`'s."""
+    ``gate``, ``slopes`` and ``chunk`` as :func:`paged_attention_plain`'s."""
     tokens = q.shape[0]
     dv = int(v_head_dim or head_dim)
     splits, per = attn_decode_plan(tokens, num_heads, num_kv_heads, max_keys, sms=sm_count(q.device))
@@ -1130,11 +1213,11 @@ def attn_decode(q, cache, table, seq_rows, token_seq, positions, out, *, num_hea
     if splits > 1:
         part_o = torch.empty(tokens * num_heads * splits * dv, dtype=torch.float32, device=q.device)
         part_ml = torch.empty(tokens * num_heads * splits * 2, dtype=torch.float32, device=q.device)
-    _check(_fn("se_attn_decode", "pppipppppp" "iiiiii" "f" "iii" "ip" "i" "fipi" "pip" "p")(
+    _check(_fn("se_attn_decode", "pppipppppp" "iiiiii" "f" "iii" "ip" "i" "fipi" "pipi" "p")(
         _ptr(q, torch.bfloat16, "q"), _ptr(cache, torch.bfloat16, "cache"), _ptr(table, torch.int32, "table"),
         table.shape[1], _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(token_seq, torch.int32, "token_seq"),
         _ptr(positions, torch.int32, "positions"), _ptr(out, torch.bfloat16, "out"), _ptr(part_o), _ptr(part_ml),
-        tokens, num_heads, num_kv_heads, head_dim, dv, page_size, float(scale), int(window or 0), splits, per,
+        tokens, num_heads, num_kv_heads, head_dim, dv, page_size, float(scale), _visible_arg(window, chunk), splits, per,
         cache.shape[0] if num_pages is None else int(num_pages), _ptr(error_word(q.device)),
         int(bool(step_inputs_settled)), *_softmax_options(q, gate, num_heads, dv, softcap, sink, keep_first or 0, slopes),
         _stream()), "attn_decode")
@@ -1143,13 +1226,13 @@ def attn_decode(q, cache, table, seq_rows, token_seq, positions, out, *, num_hea
 
 def attn_prefill(q, cache, table, seq_rows, cu_q, kv_len, out, *, entries, max_q_len, num_heads, num_kv_heads,
                  head_dim, page_size, scale, window=None, num_pages=None, v_head_dim=None, softcap=None,
-                 sink=False, gate=None, keep_first: int = 0, slopes=None):
+                 sink=False, gate=None, keep_first: int = 0, slopes=None, chunk=None):
     dv = int(v_head_dim or head_dim)
-    _check(_fn("se_attn_prefill", "pppipppp" "iiiiiii" "f" "i" "ip" "fipi" "pip" "p")(
+    _check(_fn("se_attn_prefill", "pppipppp" "iiiiiii" "f" "i" "ip" "fipi" "pipi" "p")(
         _ptr(q, torch.bfloat16, "q"), _ptr(cache, torch.bfloat16, "cache"), _ptr(table, torch.int32, "table"),
         table.shape[1], _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(cu_q, torch.int32, "cu_q"),
         _ptr(kv_len, torch.int32, "kv_len"), _ptr(out, torch.bfloat16, "out"), entries, max_q_len, num_heads,
-        num_kv_heads, head_dim, dv, page_size, float(scale), int(window or 0),
+        num_kv_heads, head_dim, dv, page_size, float(scale), _visible_arg(window, chunk),
         cache.shape[0] if num_pages is None else int(num_pages), _ptr(error_word(q.device)),
         *_softmax_options(q, gate, num_heads, dv, softcap, sink, keep_first or 0, slopes), _stream()), "attn_prefill")
     return out
@@ -1162,15 +1245,15 @@ def attn_prefill_tc_supported(head_dim: int, num_heads: int, num_kv_heads: int) 
 
 def attn_prefill_tc(q, cache, table, seq_rows, cu_q, kv_len, out, *, entries, max_q_len, num_heads, num_kv_heads,
                     head_dim, page_size, scale, window=None, num_pages=None, v_head_dim=None, softcap=None,
-                    sink: bool = False, gate=None, keep_first: int = 0, slopes=None):
+                    sink: bool = False, gate=None, keep_first: int = 0, slopes=None, chunk=None):
     """Prompt-portion attention on tcgen05 (head size 128, values of the same size)."""
     if int(v_head_dim or head_dim) != head_dim:
         raise ValueError("the tcgen05 prompt kernel takes values of the keys' head size")
-    _check(_fn("se_attn_prefill_tc", "pppippppp" "iiiiii" "f" "ii" "fipi" "pip" "p")(
+    _check(_fn("se_attn_prefill_tc", "pppippppp" "iiiiii" "f" "ii" "fipi" "pipi" "p")(
         _ptr(q, torch.bfloat16, "q"), _ptr(cache, torch.bfloat16, "cache"), _ptr(table, torch.int32, "table"),
         table.shape[1], _ptr(seq_rows, torch.int32, "seq_rows"), _ptr(cu_q, torch.int32, "cu_q"),
         _ptr(kv_len, torch.int32, "kv_len"), _ptr(out, torch.bfloat16, "out"), _ptr(error_word(q.device)),
-        entries, max_q_len, num_heads, num_kv_heads, head_dim, page_size, float(scale), int(window or 0),
+        entries, max_q_len, num_heads, num_kv_heads, head_dim, page_size, float(scale), _visible_arg(window, chunk),
         cache.shape[0] if num_pages is None else int(num_pages),
         *_softmax_options(q, gate, num_heads, head_dim, softcap, sink, keep_first or 0, slopes), _stream()),
         "attn_prefill_tc")

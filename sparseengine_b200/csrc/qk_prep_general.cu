@@ -7,13 +7,15 @@
 //   K page   = rot(k * inv_rms(k) * k_w, pos)
 //   V page   = v, or (1 - mix) * v + mix * v_first              (v_first: the same token's values elsewhere)
 //   temp(p)  = 1 + coef * ln(floor((p + 1) / every) + 1)        (coef = 0: none)
-//   rot      : on the first `rotary_dim` dims of every head, dim i paired with dim i + rotary_dim/2,
-//              (u, v) -> (u cos a - v sin a, v cos a + u sin a), a = pos * inv_freq[i]  (rotary_dim = 0: none)
+//   rot      : on the first `rotary_dim` dims of every head, dim i paired with dim i + rotary_dim/2 (or, `interleaved`,
+//              dim 2i with dim 2i + 1), (u, v) -> (u cos a - v sin a, v cos a + u sin a), a = pos * inv_freq[i], cos and
+//              sin multiplied by `rope_scale`  (rotary_dim = 0: none)
 //
 // Options: `bias` (32-bit, [q | k | v] like the projection row) is added to the projection before
 // anything else; `per_head` 1 norms every head by its own root mean square, with weights of d elements
 // shared by the heads, instead of the whole projection with a weight per column; `per_head` 2 does so for
-// queries and keys without weights.
+// queries and keys without weights, and its root mean square is that of the rotated head (a rotation keeps a pair's
+// sum of squares, so the squares of the rotated dims are counted rope_scale^2 times and nothing is rotated twice).
 //
 // Everything is computed in 32-bit and rounded once.  The norm weights are
 // optional.  The projection row is [q: hq*d | k: hkv*d | v: hkv*dv] (`has_kv`) or [q] alone.
@@ -35,7 +37,7 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
                        const int* __restrict__ seq_rows, const int* __restrict__ table, int table_stride,
                        T* __restrict__ cache, T* __restrict__ q_out, int hq, int hkv, int d, int dv, float eps,
                        float temp_coef, int temp_every, int page_size, int has_kv, int num_pages, int* __restrict__ error,
-                       const float* __restrict__ bias, int per_head) {
+                       const float* __restrict__ bias, int per_head, int interleaved, float rope_scale) {
     extern __shared__ float inv_head[];      // per_head: the inverse root mean square of every q head, then every k head
     __shared__ float scratch[33];
     grid_dependency_trigger();
@@ -54,7 +56,7 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
     const int half = rotary_dim / 2;
     const T* vf = v_first != nullptr ? v_first + (size_t)t * v_first_pitch : nullptr;
     // Eight elements at a time where sizes and addresses allow it.
-    const bool vec = (d & 7) == 0 && (half & 7) == 0 && (dv & 7) == 0 && (pitch & 7) == 0 && aligned8(proj) && aligned8(q_out) &&
+    const bool vec = (d & 7) == 0 && (interleaved ? (rotary_dim & 7) == 0 : (half & 7) == 0) && (dv & 7) == 0 && (pitch & 7) == 0 && aligned8(proj) && aligned8(q_out) &&
                      (bias == nullptr || aligned8(bias)) &&
                      (q_w == nullptr || aligned8(q_w)) && (k_w == nullptr || aligned8(k_w)) && (cache == nullptr || aligned8(cache)) &&
                      (vf == nullptr || ((v_first_pitch & 7) == 0 && aligned8(v_first)));
@@ -95,7 +97,8 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
             if (normed) {
                 const T* part = is_q ? row + (size_t)h * d : row + qn + (size_t)(h - hq) * d;
                 const int b0 = is_q ? h * d : qn + (h - hq) * d;
-                for (int i = lane; i < d; i += 32) { const float v = raw(part, b0, i); ss += v * v; }
+                const float rot2 = per_head == 2 ? rope_scale * rope_scale : 1.f;
+                for (int i = lane; i < d; i += 32) { const float v = raw(part, b0, i); ss += i < rotary_dim ? rot2 * v * v : v * v; }
                 ss = warp_sum(ss);
             }
             if (lane == 0) inv_head[h] = normed ? 1.0f / sqrtf(ss / (float)d + eps) : 1.f;
@@ -107,7 +110,12 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
     }
     // cos and sin of the token's angles, once for all heads
     __shared__ float cs_t[kMaxHalf], sn_t[kMaxHalf];
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &sn_t[i], &cs_t[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, cs;
+        sincosf((float)pos * inv_freq[i], &sn, &cs);
+        sn_t[i] = sn * rope_scale;
+        cs_t[i] = cs * rope_scale;
+    }
     __syncthreads();
     T* kbase = nullptr;
     T* vbase = nullptr;
@@ -122,7 +130,7 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
     // The 8-wide path: a work item is a pair of 8-element chunks that rotate into one another (columns c
     // and c + half of a head), or one chunk that passes.
     if (vec) {
-        const int pair_items = half / 8, items = d / 8 - pair_items;          // per head
+        const int pair_items = interleaved ? 0 : half / 8, items = d / 8 - pair_items;          // per head
         auto normed8 = [&](const T* part, int b0, const T* w, float inv, int i, int wi, float* v) {
             raw8(part, b0, i, v);
 #pragma unroll
@@ -161,8 +169,16 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
                 store8(dst + c, ra);
                 store8(dst + c + half, rb);
             } else {
-                const int c = rotary_dim + (k - pair_items) * 8;
+                const int c = interleaved ? k * 8 : rotary_dim + (k - pair_items) * 8;
                 normed8(part, b0, w, inv, hh * d + c, w0 + c, a);
+                if (interleaved && c < rotary_dim) {
+#pragma unroll
+                    for (int j = 0; j < 8; j += 2) {
+                        const float cs = cs_t[(c + j) / 2], sn = sn_t[(c + j) / 2], u = a[j], v = a[j + 1];
+                        a[j] = u * cs - v * sn;
+                        a[j + 1] = v * cs + u * sn;
+                    }
+                }
 #pragma unroll
                 for (int j = 0; j < 8; ++j) a[j] *= mul;
                 store8(dst + c, a);
@@ -196,11 +212,13 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
         float v = raw(part, b0, i) * inv;
         if (w != nullptr) v *= to_float(w[per_head ? c : i]);
         if (c >= rotary_dim) return v;
-        const int j = c < half ? i + half : i - half;
+        const bool first = interleaved ? (c & 1) == 0 : c < half;
+        const int step = interleaved ? 1 : half, j = first ? i + step : i - step;
+        const int pair = interleaved ? c / 2 : first ? c : c - half;
         float u = raw(part, b0, j) * inv;
         if (w != nullptr) u *= to_float(w[per_head ? j % d : j]);
-        const float sn = sn_t[c < half ? c : c - half], cs = cs_t[c < half ? c : c - half];
-        return c < half ? v * cs - u * sn : v * cs + u * sn;
+        const float sn = sn_t[pair], cs = cs_t[pair];
+        return first ? v * cs - u * sn : v * cs + u * sn;
     };
     for (int i = threadIdx.x; i < qn; i += blockDim.x)
         qdst[i] = from_float<T>(prepared(row, 0, q_w, inv_q, 0, i) * temp);
@@ -217,52 +235,111 @@ qk_prep_general_kernel(const T* proj, int pitch, const T* __restrict__ q_w, cons
     }
 }
 
-// Per-head norms (per_head 1 with weights, 2 without) and nothing else: no rotation, temperature, bias or blending.
-// Every 16-byte chunk (float32: two) of the step's projection rows is a lane's work item; a head's LANES = d / 8
-// chunks lie in neighbouring lanes of one warp, so its sum of squares is a few shuffles and each input is read once.
-template <typename T, int LANES>
-__global__ void __launch_bounds__(256)
+// Per-head work and nothing else: biases, per-head norms (NORM 1 with weights, 2 without, 0 none) and a rotation (ROT 1
+// split halves, 2 neighbours, 0 none); no temperature and no blending.  Every 16-byte chunk (float32: two) of the step's
+// projection rows is a lane's work item.  With norms a head's d / 8 chunks lie in neighbouring lanes of one warp (d / 8 a
+// power of two), so its sum of squares is a few shuffles; split halves read the partner's chunk once more.  Cosines
+// and sines of the tokens a block meets are worked out once, in shared memory.
+constexpr int kPrepItems = 256;      // work items (threads) of a block
+__host__ __device__ __forceinline__ int prep_block_tokens(int per_token) { return kPrepItems / per_token + 2; }
+
+template <typename T, int NORM, int ROT>
+__global__ void __launch_bounds__(kPrepItems)
 qk_prep_heads_kernel(const T* proj, int pitch, const T* __restrict__ q_w, const T* __restrict__ k_w,
+                     const float* __restrict__ inv_freq, int rotary_dim, float rope_scale, const float* __restrict__ bias,
                      const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ seq_rows,
                      const int* __restrict__ table, int table_stride, T* cache, T* q_out, long long items, int hq, int hkv,
-                     int dv, float eps, int page_size, int num_pages, int* __restrict__ error) {
-    constexpr int d = 8 * LANES;
+                     int d, int dv, float eps, int page_size, int num_pages, int* __restrict__ error) {
+    extern __shared__ float2 turns[];            // [tokens of the block][rotary_dim / 2]: (cos, sin) * rope_scale
     grid_dependency_trigger();
+    const int lanes = d / 8, qc = hq * lanes, kc = hkv * lanes, per_token = qc + kc + hkv * (dv / 8);
+    const long long x0 = (long long)blockIdx.x * kPrepItems, x = x0 + threadIdx.x;
+    const int t_first = (int)(x0 / per_token), half = rotary_dim / 2;
     grid_dependency_wait();
-    const int qc = hq * LANES, kc = hkv * LANES, per_token = qc + kc + hkv * (dv / 8);
-    const long long x = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    const bool live = x < items;
-    const int t = live ? (int)(x / per_token) : 0;
-    const int c = live ? (int)(x - (long long)t * per_token) : 0;
-    float v[8];
-    load8(proj + (size_t)t * pitch + 8 * c, v);
-    float ss = 0.f;
-#pragma unroll
-    for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
-#pragma unroll
-    for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);       // items of values: a sum nobody uses
-    if (!live) return;
-    const int in_head = (c % LANES) * 8;
-    if (c < qc + kc) {
-        const T* w = c < qc ? q_w : k_w;
-        const float inv = 1.0f / sqrtf(ss / (float)d + eps);
-        float wv[8];
-        if (w != nullptr) load8(w + in_head, wv);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) v[j] *= w != nullptr ? inv * wv[j] : inv;
+    if (ROT) {
+        const long long last = x0 + kPrepItems - 1 < items ? x0 + kPrepItems - 1 : items - 1;
+        const int n = ((int)(last / per_token) - t_first + 1) * half;
+        for (int i = threadIdx.x; i < n; i += kPrepItems) {
+            const int t = i / half;
+            float sn, cs;
+            sincosf((float)positions[t_first + t] * inv_freq[i - t * half], &sn, &cs);
+            turns[i] = make_float2(cs * rope_scale, sn * rope_scale);
+        }
     }
-    if (c < qc) {
-        store8(q_out + ((size_t)t * qc + c) * 8, v);
-        return;
+    const bool live = x < items;
+    const int t = live ? (int)(x / per_token) : t_first;
+    const int c = live ? (int)(x - (long long)t * per_token) : 0;
+    const T* row = proj + (size_t)t * pitch;
+    auto load_raw = [&](int chunk, float* v) {
+        load8(row + 8 * chunk, v);
+        if (bias != nullptr) {
+            float b[8];
+            load8(bias + 8 * chunk, b);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] += b[j];
+        }
+    };
+    float v[8];
+    load_raw(c, v);
+    const bool is_q = c < qc, is_v = c >= qc + kc;
+    const int head = is_v ? 0 : c / lanes;
+    const int in_head = is_v ? 0 : (c - head * lanes) * 8;
+    float inv = 1.f;
+    if (NORM) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+        // a chunk rotates as a whole or not at all (rotary_dim a multiple of 8)
+        if (NORM == 2 && ROT && in_head < rotary_dim) ss *= rope_scale * rope_scale;
+        for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);       // items of values: a sum nobody uses
+        inv = 1.0f / sqrtf(ss / (float)d + eps);
+    }
+    if (ROT) __syncthreads();
+    if (!live) return;
+    if (!is_v) {
+        const T* w = is_q ? q_w : k_w;
+        auto weigh = [&](int at, float* a) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) a[j] *= inv;
+            if (NORM == 1) {
+                float wv[8];
+                load8(w + at, wv);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) a[j] *= wv[j];
+            }
+        };
+        if (NORM) weigh(in_head, v);
+        if (ROT == 1 && in_head < rotary_dim) {
+            const bool first = in_head < half;
+            const int other = first ? in_head + half : in_head - half;
+            float u[8];
+            load_raw(head * lanes + other / 8, u);
+            if (NORM) weigh(other, u);
+            const float2* cs = turns + (size_t)(t - t_first) * half + (first ? in_head : other);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = first ? v[j] * cs[j].x - u[j] * cs[j].y : v[j] * cs[j].x + u[j] * cs[j].y;
+        }
+        if (ROT == 2 && in_head < rotary_dim) {
+            const float2* cs = turns + (size_t)(t - t_first) * half + in_head / 2;
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                const float a = v[j], b = v[j + 1];
+                v[j] = a * cs[j / 2].x - b * cs[j / 2].y;
+                v[j + 1] = b * cs[j / 2].x + a * cs[j / 2].y;
+            }
+        }
+        if (is_q) {
+            store8(q_out + ((size_t)t * qc + c) * 8, v);
+            return;
+        }
     }
     const int pos = positions[t];
     const int page = table[(size_t)seq_rows[token_seq[t]] * table_stride + pos / page_size];
     if (!page_in_pool(page, num_pages, error, SE_CODE_BAD_PAGE_QK_PREP)) return;
     const int slot = pos % page_size;
     T* base = cache + (size_t)page * hkv * page_size * (d + dv);
-    if (c < qc + kc) {
-        const int h = (c - qc) / LANES;
-        store8(base + ((size_t)h * page_size + slot) * d + in_head, v);
+    if (!is_v) {
+        store8(base + ((size_t)(head - hq) * page_size + slot) * d + in_head, v);
     } else {
         const int i = (c - qc - kc) * 8, h = i / dv;
         store8(base + (size_t)hkv * page_size * d + ((size_t)h * page_size + slot) * dv + (i - h * dv), v);
@@ -277,33 +354,42 @@ extern "C" int se_qk_prep_general(const void* proj, int pitch, const void* q_w, 
                                   const int* token_seq, const int* seq_rows, const int* table, int table_stride,
                                   void* cache, void* q_out, int tokens, int hq, int hkv, int d, int dv, float eps,
                                   float temp_coef, int temp_every, int page_size, int has_kv, int num_pages, int* error,
-                                  const float* bias, int per_head, int dtype, cudaStream_t stream) {
+                                  const float* bias, int per_head, int interleaved, float rope_scale, int dtype,
+                                  cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (hq <= 0 || d <= 0 || (has_kv && (hkv <= 0 || dv <= 0 || page_size <= 0))) return SE_ERR_ARGUMENT;
     if (pitch < hq * d + (has_kv ? hkv * (d + dv) : 0)) return SE_ERR_ARGUMENT;
     if (rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) || (rotary_dim > 0 && inv_freq == nullptr)) return SE_ERR_ARGUMENT;
     if (rotary_dim > 2 * se::kMaxHalf) return SE_ERR_UNSUPPORTED;
+    if (rotary_dim == 0) rope_scale = 1.f;
     if (v_first != nullptr && (v_mix == nullptr || !has_kv || v_first_pitch < hkv * dv)) return SE_ERR_ARGUMENT;
-    // heads of 64, 128 or 256 elements that are normed and nothing else
+    // per-head work alone, in chunks of 8 elements
     const size_t esize = dtype == SE_DTYPE_F32 ? 4 : 2;
-    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    const int lanes = d / 8;
-    if (has_kv && per_head && rotary_dim == 0 && (temp_coef == 0.f || temp_every <= 0) && v_first == nullptr && bias == nullptr &&
-        (per_head == 2 || (q_w != nullptr && k_w != nullptr)) && (d == 64 || d == 128 || d == 256) && (dv & 7) == 0 &&
-        (hkv * (dv / 8)) % lanes == 0 && (pitch * esize) % 16 == 0 && aligned(proj) && aligned(q_out) && aligned(cache) &&
-        (q_w == nullptr || aligned(q_w)) && (k_w == nullptr || aligned(k_w))) {
-        const long long items = (long long)tokens * ((hq + hkv) * lanes + hkv * (dv / 8));
-        const long long blocks = (items + 255) / 256;
+    auto aligned = [](const void* p) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int lanes = d / 8, per_token = hkv > 0 ? (hq + hkv) * lanes + hkv * (dv / 8) : 0;
+    const bool normed = per_head != 0, lanes_fit = lanes >= 1 && lanes <= 32 && (lanes & (lanes - 1)) == 0 && (hkv * (dv / 8)) % lanes == 0;
+    if (has_kv && (normed ? lanes_fit && (per_head == 2 || (q_w != nullptr && k_w != nullptr)) : q_w == nullptr && k_w == nullptr) &&
+        (normed || rotary_dim > 0 || bias != nullptr) && (temp_coef == 0.f || temp_every <= 0) && v_first == nullptr && (d & 7) == 0 && (dv & 7) == 0 &&
+        (interleaved ? (rotary_dim & 7) == 0 : (rotary_dim & 15) == 0) && (pitch * esize) % 16 == 0 && aligned(proj) &&
+        aligned(q_out) && aligned(cache) && aligned(q_w) && aligned(k_w) && aligned(bias)) {
+        const long long items = (long long)tokens * per_token;
+        const long long blocks = (items + se::kPrepItems - 1) / se::kPrepItems;
         if (blocks > 0x7fffffffLL) return SE_ERR_UNSUPPORTED;
-        const bool weights = per_head == 1;
+        const size_t turns = rotary_dim > 0 ? (size_t)se::prep_block_tokens(per_token) * (rotary_dim / 2) * sizeof(float2) : 0;
+        const int norm = per_head, rot = rotary_dim == 0 ? 0 : interleaved ? 2 : 1;
+#define SE_PREP_CASE(N, R)                                                                                                  \
+    if (norm == N && rot == R)                                                                                              \
+        e = SE_LAUNCH_DEPENDENT("qk", (se::qk_prep_heads_kernel<T, N, R>), dim3((unsigned)blocks), dim3(se::kPrepItems), turns, stream, \
+                                 (const T*)proj, pitch, (const T*)q_w, (const T*)k_w, inv_freq, rotary_dim, rope_scale, bias, \
+                                 positions, token_seq, seq_rows, table, table_stride, (T*)cache, (T*)q_out, items, hq, hkv, d, \
+                                 dv, eps, page_size, num_pages, error);
         SE_DISPATCH_DTYPE(dtype, T, {
-            auto kernel = d == 64 ? se::qk_prep_heads_kernel<T, 8> : d == 128 ? se::qk_prep_heads_kernel<T, 16> : se::qk_prep_heads_kernel<T, 32>;
-            cudaError_t e = SE_LAUNCH_DEPENDENT("qk", kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, pitch,
-                                                 weights ? (const T*)q_w : nullptr, weights ? (const T*)k_w : nullptr, positions,
-                                                 token_seq, seq_rows, table, table_stride, (T*)cache, (T*)q_out, items, hq, hkv, dv,
-                                                 eps, page_size, num_pages, error);
+            cudaError_t e = cudaErrorInvalidValue;
+            SE_PREP_CASE(0, 0) SE_PREP_CASE(0, 1) SE_PREP_CASE(0, 2) SE_PREP_CASE(1, 0) SE_PREP_CASE(1, 1) SE_PREP_CASE(1, 2)
+            SE_PREP_CASE(2, 0) SE_PREP_CASE(2, 1) SE_PREP_CASE(2, 2)
             if (e != cudaSuccess) return (int)e;
         });
+#undef SE_PREP_CASE
         SE_LAUNCH_CHECK();
     }
     const size_t smem = per_head ? (size_t)(hq + (has_kv ? hkv : 0)) * sizeof(float) : 0;
@@ -313,7 +399,7 @@ extern "C" int se_qk_prep_general(const void* proj, int pitch, const void* q_w, 
                                              (const T*)proj, pitch, (const T*)q_w, (const T*)k_w, inv_freq, rotary_dim, (const T*)v_first,
                                              v_first_pitch, v_mix, positions, token_seq, seq_rows,
                                              table, table_stride, (T*)cache, (T*)q_out, hq, hkv, d, dv, eps, temp_coef, temp_every,
-                                             page_size, has_kv, num_pages, error, bias, per_head);
+                                             page_size, has_kv, num_pages, error, bias, per_head, interleaved, rope_scale);
         if (e != cudaSuccess) return (int)e;
     });
     SE_LAUNCH_CHECK();

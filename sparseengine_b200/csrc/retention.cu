@@ -5,7 +5,9 @@
 //
 // q and k are rotated by their position on the first `rotary_dim` dims of each head (dim i pairs
 // with i + rotary_dim/2, angle = position * inv_freq[i]); k is multiplied by `k_scale` after the
-// rotation.  Each head's o is divided by its root mean square and multiplied by silu(gate).
+// rotation.  Each head's o is divided by its root mean square and multiplied by silu(gate); or (`joint`) the
+// concatenated heads are divided by one root mean square, multiplied by a weight per column and by sigmoid(gate).
+// With `silu` q, k and v are silu of the projection (before any rotation or factor).
 // Rotation, scaling, state, sums and the norm are 32-bit; q, k, v and the gate come from the
 // projection in the activation type.
 //
@@ -15,12 +17,19 @@
 
 namespace se {
 
+__device__ __forceinline__ float silu32(float v) { return v / (1.f + expf(-v)); }
+// values that came from 16 bits: the fast exponential and quotient (a few units in the last place of 32-bit)
+template <typename T> __device__ __forceinline__ float input_silu(float v) {
+    return sizeof(T) == 2 ? __fdividef(v, 1.f + __expf(-v)) : silu32(v);
+}
+
 // q32, k32 [tokens, heads, d]: rotated (k also scaled), 32-bit.  One thread per (token, head, dim).
 template <typename T>
 __global__ void retention_prep_kernel(const T* proj, int proj_stride, int q_off, int k_off,
                                       const float* __restrict__ inv_freq, const int* __restrict__ positions,
                                       float* __restrict__ q32, float* __restrict__ k32, int tokens, int heads, int d,
-                                      int rotary_dim, float k_scale) {
+                                      int rotary_dim, float k_scale, int silu) {
+    auto in = [&](T v) { const float f = to_float(v); return silu ? input_silu<T>(f) : f; };
     const size_t n = (size_t)tokens * heads * d;
     const int half = rotary_dim / 2;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x) {
@@ -29,13 +38,13 @@ __global__ void retention_prep_kernel(const T* proj, int proj_stride, int q_off,
         const int t = (int)(idx / ((size_t)d * heads));
         const T* qp = proj + (size_t)t * proj_stride + q_off + h * d;
         const T* kp = proj + (size_t)t * proj_stride + k_off + h * d;
-        float qv = to_float(qp[i]), kv = to_float(kp[i]);
+        float qv = in(qp[i]), kv = in(kp[i]);
         if (i < rotary_dim) {
             const int j = i < half ? i : i - half;
             float sn, cs;
             sincosf((float)positions[t] * inv_freq[j], &sn, &cs);
-            const float qu = to_float(qp[j]), qw = to_float(qp[j + half]);
-            const float ku = to_float(kp[j]), kw = to_float(kp[j + half]);
+            const float qu = in(qp[j]), qw = in(qp[j + half]);
+            const float ku = in(kp[j]), kw = in(kp[j + half]);
             qv = i < half ? qu * cs - qw * sn : qw * cs + qu * sn;
             kv = i < half ? ku * cs - kw * sn : kw * cs + ku * sn;
         }
@@ -44,18 +53,39 @@ __global__ void retention_prep_kernel(const T* proj, int proj_stride, int q_off,
     }
 }
 
+// The same without a rotation, eight neighbours at a time (heads * d a multiple of 8, 16-byte rows).
+template <typename T>
+__global__ void retention_prep8_kernel(const T* proj, int proj_stride, int q_off, int k_off, float* __restrict__ q32,
+                                       float* __restrict__ k32, int tokens, int chunks, float k_scale, int silu) {
+    grid_dependency_trigger();
+    grid_dependency_wait();
+    const size_t n = (size_t)tokens * 2 * chunks;
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x) {
+        const int t = (int)(idx / (2 * chunks)), c = (int)(idx - (size_t)t * 2 * chunks);
+        const bool is_k = c >= chunks;
+        const int i = (is_k ? c - chunks : c) * 8;
+        float v[8];
+        load8(proj + (size_t)t * proj_stride + (is_k ? k_off : q_off) + i, v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = (silu ? input_silu<T>(v[j]) : v[j]) * (is_k ? k_scale : 1.f);
+        store8((is_k ? k32 : q32) + (size_t)t * chunks * 8 + i, v);
+    }
+}
+
 constexpr int kRetWarps = 8;        // the state's rows are dealt to the warps: warp r holds rows r, r + 8, ...
 constexpr int kRetTokens = 8;       // tokens staged at a time
 
 // One block per (entry, head, 32 value columns).  Thread (warp r, lane c) keeps rows r + 8 n of column
 // c in registers; a token's partial sums over a warp's rows meet in shared memory, eight tokens at
-// a time.  Sums run in one fixed order whatever the batch or the portion.
+// a time.  Sums run in one fixed order whatever the batch or the portion.  Without q32 and k32 (nullptr) q and k are
+// read from the projection as they are staged (no rotation): silu of it with `silu`, k times k_scale.
 template <typename T, int NPT>
 __global__ void __launch_bounds__(32 * kRetWarps)
 retention_scan_kernel(const float* __restrict__ q32, const float* __restrict__ k32, const T* proj, int proj_stride,
                       int v_off, const float* __restrict__ decay, float* state, long long state_stride,
                       const int* __restrict__ cu_q, const int* __restrict__ seq_rows, float* __restrict__ o, int heads,
-                      int d, int dv) {
+                      int d, int dv, int silu, int q_off, int k_off, float k_scale) {
+    grid_dependency_trigger();
     extern __shared__ float ret_smem[];
     float* qs = ret_smem;                                   // [kRetTokens][d]
     float* ks = qs + kRetTokens * d;                        // [kRetTokens][d]
@@ -70,23 +100,34 @@ retention_scan_kernel(const float* __restrict__ q32, const float* __restrict__ k
     const float g = decay[h];
     float* S = state + (size_t)seq_rows[s] * state_stride + (size_t)h * d * dv;
     float st[NPT];
+    // The state was last written by an earlier step, which the kernel before this one has seen the end of: it is read
+    // while that kernel (the one that makes the projection) may still run.  The step's tensors are older as well.
 #pragma unroll
     for (int n = 0; n < NPT; ++n) {
         const int i = warp + kRetWarps * n;
         st[n] = (i < d && col_ok) ? S[(size_t)i * dv + col] : 0.f;
     }
+    grid_dependency_wait();
     for (int tb = t0; tb < t1; tb += kRetTokens) {
         const int nt = min(kRetTokens, t1 - tb);
         __syncthreads();                                    // the last round's sums have been read
         for (int x = threadIdx.x; x < nt * d; x += blockDim.x) {
             const int tt = x / d, i = x - tt * d;
-            const size_t at = ((size_t)(tb + tt) * heads + h) * d + i;
-            qs[tt * d + i] = q32[at];
-            ks[tt * d + i] = k32[at];
+            if (q32 != nullptr) {
+                const size_t at = ((size_t)(tb + tt) * heads + h) * d + i;
+                qs[tt * d + i] = q32[at];
+                ks[tt * d + i] = k32[at];
+            } else {
+                const T* row = proj + (size_t)(tb + tt) * proj_stride + h * d + i;
+                const float qv = to_float(row[q_off]), kv = to_float(row[k_off]);
+                qs[tt * d + i] = silu ? input_silu<T>(qv) : qv;
+                ks[tt * d + i] = (silu ? input_silu<T>(kv) : kv) * k_scale;
+            }
         }
         for (int x = threadIdx.x; x < nt * 32; x += blockDim.x) {
             const int tt = x >> 5, c = x & 31;
-            vs[x] = c0 + c < dv ? to_float(proj[(size_t)(tb + tt) * proj_stride + v_off + h * dv + c0 + c]) : 0.f;
+            const float v = c0 + c < dv ? to_float(proj[(size_t)(tb + tt) * proj_stride + v_off + h * dv + c0 + c]) : 0.f;
+            vs[x] = silu ? input_silu<T>(v) : v;
         }
         __syncthreads();
         for (int tt = 0; tt < nt; ++tt) {
@@ -149,7 +190,7 @@ __global__ void __launch_bounds__(kChunkThreads, 2)
 retention_chunk_kernel(const float* __restrict__ q32, const float* __restrict__ k32, const T* proj, int proj_stride,
                        int v_off, const float* __restrict__ decay, float* state, long long state_stride,
                        const int* __restrict__ cu_q, const int* __restrict__ seq_rows, float* __restrict__ o, int heads,
-                       int d, int dv, int max_seg, int seg_len, float* __restrict__ seg_state) {
+                       int d, int dv, int max_seg, int seg_len, float* __restrict__ seg_state, int silu) {
     extern __shared__ __align__(16) float chunk_smem[];
     float* qs = chunk_smem;                      // [d][kPitch]
     float* ks = qs + d * kPitch;                 // [d][kPitch]
@@ -194,7 +235,8 @@ retention_chunk_kernel(const float* __restrict__ q32, const float* __restrict__ 
         asm volatile("cp.async.commit_group;" ::: "memory");
         for (int x = threadIdx.x; x < kChunk * 32; x += kChunkThreads) {
             const int t = x >> 5, c = x & 31;
-            vs[x] = (t < n && c0 + c < dv) ? to_float(proj[(size_t)(tb + t) * proj_stride + v_off + h * dv + c0 + c]) : 0.f;
+            const float v = (t < n && c0 + c < dv) ? to_float(proj[(size_t)(tb + t) * proj_stride + v_off + h * dv + c0 + c]) : 0.f;
+            vs[x] = silu ? input_silu<T>(v) : v;
         }
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
@@ -369,39 +411,118 @@ __global__ void retention_out_kernel(const float* __restrict__ o, const T* proj,
     }
 }
 
+// out[t, :] = o[t, :] / sqrt(mean(o[t, :]^2) + eps) * w * sigmoid(gate[t, :]) over the concatenated heads (`width`
+// columns); a block per token, each thread keeps what it has read in registers where the row is short enough.
+constexpr int kJointKeep = 4;        // chunks of 8 columns a thread keeps
+template <typename T>
+__global__ void retention_out_joint_kernel(const float* o, const T* proj, int proj_stride, int g_off, const T* __restrict__ w,
+                                           T* __restrict__ out, int width, float eps, int vec) {
+    __shared__ float scratch[33];
+    grid_dependency_trigger();
+    grid_dependency_wait();
+    const float* op = o + (size_t)blockIdx.x * width;
+    const T* gp = proj + (size_t)blockIdx.x * proj_stride + g_off;
+    T* dst = out + (size_t)blockIdx.x * width;
+    float ss = 0.f;
+    if (!vec) {
+        for (int i = threadIdx.x; i < width; i += blockDim.x) ss += op[i] * op[i];
+        const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+        for (int i = threadIdx.x; i < width; i += blockDim.x)
+            dst[i] = from_float<T>(op[i] * inv * to_float(w[i]) / (1.f + expf(-to_float(gp[i]))));
+        return;
+    }
+    float keep[kJointKeep][8], gate[kJointKeep][8];
+    const int step = blockDim.x * 8;
+#pragma unroll
+    for (int k = 0; k < kJointKeep; ++k) {
+        const int i = threadIdx.x * 8 + k * step;
+        if (i < width) {
+            load8(op + i, keep[k]);
+            load8(gp + i, gate[k]);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss += keep[k][j] * keep[k][j];
+        }
+    }
+    for (int i = threadIdx.x * 8 + kJointKeep * step; i < width; i += step) {
+        float v[8];
+        load8(op + i, v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+    auto finish = [&](int i, float* v, const float* g) {
+        float wv[8];
+        load8(w + i, wv);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float y = v[j] * inv * wv[j];
+            v[j] = sizeof(T) == 2 ? __fdividef(y, 1.f + __expf(-g[j])) : y / (1.f + expf(-g[j]));
+        }
+        store8(dst + i, v);
+    };
+#pragma unroll
+    for (int k = 0; k < kJointKeep; ++k) {
+        const int i = threadIdx.x * 8 + k * step;
+        if (i < width) finish(i, keep[k], gate[k]);
+    }
+    for (int i = threadIdx.x * 8 + kJointKeep * step; i < width; i += step) {
+        float v[8], g[8];
+        load8(op + i, v);
+        load8(gp + i, g);
+        finish(i, v, g);
+    }
+}
+
 }  // namespace se
 
 extern "C" int se_retention_max_head_dim() { return se::kRetWarps * 32; }
 
 extern "C" int se_retention_prep(const void* proj, int proj_stride, int q_off, int k_off, const float* inv_freq,
                                  const int* positions, float* q32, float* k32, int tokens, int heads, int d,
-                                 int rotary_dim, float k_scale, int dtype, cudaStream_t stream) {
+                                 int rotary_dim, float k_scale, int silu, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (heads <= 0 || d <= 0 || rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1)) return SE_ERR_ARGUMENT;
+    const size_t esize = dtype == SE_DTYPE_F32 ? 4 : 2;
+    if (rotary_dim == 0 && (heads * d) % 8 == 0 && (proj_stride * esize) % 16 == 0 && (q_off * esize) % 16 == 0 &&
+        (k_off * esize) % 16 == 0 && ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q32) | reinterpret_cast<uintptr_t>(k32)) & 15) == 0) {
+        const int chunks = heads * d / 8;
+        const long long items = (long long)tokens * 2 * chunks;
+        const int grid = (int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16);
+        SE_DISPATCH_DTYPE(dtype, T, {
+            cudaError_t e = SE_LAUNCH_DEPENDENT("ret", se::retention_prep8_kernel<T>, dim3(grid), dim3(256), 0, stream, (const T*)proj,
+                                                 proj_stride, q_off, k_off, q32, k32, tokens, chunks, k_scale, silu);
+            if (e != cudaSuccess) return (int)e;
+        });
+        SE_LAUNCH_CHECK();
+    }
     const long long n = (long long)tokens * heads * d;
     const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
     SE_DISPATCH_DTYPE(dtype, T,
         se::retention_prep_kernel<T><<<blocks, 256, 0, stream>>>((const T*)proj, proj_stride, q_off, k_off, inv_freq,
-                                                                  positions, q32, k32, tokens, heads, d, rotary_dim, k_scale));
+                                                                  positions, q32, k32, tokens, heads, d, rotary_dim, k_scale, silu));
     SE_LAUNCH_CHECK();
 }
 
 extern "C" int se_retention_scan(const float* q32, const float* k32, const void* proj, int proj_stride, int v_off,
                                  const float* decay, float* state, long long state_stride, const int* cu_q,
-                                 const int* seq_rows, float* o, int entries, int heads, int d, int dv, int dtype,
-                                 cudaStream_t stream) {
+                                 const int* seq_rows, float* o, int entries, int heads, int d, int dv, int silu, int q_off,
+                                 int k_off, float k_scale, int dtype, cudaStream_t stream) {
+    // q32 and k32 nullptr: q and k come from the projection's columns q_off and k_off, unrotated
     if (entries <= 0) return 0;
     if (d <= 0 || d > se_retention_max_head_dim() || dv <= 0 || heads <= 0 || heads > 65535 || (dv + 31) / 32 > 65535)
         return SE_ERR_UNSUPPORTED;
     dim3 grid(entries, heads, (dv + 31) / 32);
     const size_t smem = (size_t)(2 * se::kRetTokens * d + se::kRetTokens * 32 + se::kRetTokens * se::kRetWarps * 32) * sizeof(float);
 #define SE_RET_LAUNCH(NPT)                                                                                          \
-    se::retention_scan_kernel<T, NPT><<<grid, 32 * se::kRetWarps, smem, stream>>>(                                  \
-        q32, k32, (const T*)proj, proj_stride, v_off, decay, state, state_stride, cu_q, seq_rows, o, heads, d, dv)
+    e = SE_LAUNCH_DEPENDENT("ret", (se::retention_scan_kernel<T, NPT>), grid, dim3(32 * se::kRetWarps), smem, stream,     \
+                             q32, k32, (const T*)proj, proj_stride, v_off, decay, state, state_stride, cu_q, seq_rows, o,   \
+                             heads, d, dv, silu, q_off, k_off, k_scale)
     SE_DISPATCH_DTYPE(dtype, T, {
+        cudaError_t e = cudaSuccess;
         if (d <= 8 * se::kRetWarps) SE_RET_LAUNCH(8);
         else if (d <= 16 * se::kRetWarps) SE_RET_LAUNCH(16);
         else SE_RET_LAUNCH(32);
+        if (e != cudaSuccess) return (int)e;
     });
 #undef SE_RET_LAUNCH
     SE_LAUNCH_CHECK();
@@ -413,7 +534,7 @@ extern "C" int se_retention_chunk_supported(int d) { return d > 0 && d <= 256; }
 extern "C" int se_retention_chunk(const float* q32, const float* k32, const void* proj, int proj_stride, int v_off,
                                   const float* decay, float* state, long long state_stride, const int* cu_q,
                                   const int* seq_rows, float* o, int entries, int heads, int d, int dv, int max_seg,
-                                  int seg_len, float* seg_state, int dtype, cudaStream_t stream) {
+                                  int seg_len, float* seg_state, int silu, int dtype, cudaStream_t stream) {
     // max_seg > 1: the entries' tokens in segments of seg_len (a multiple of 64) that run side by side, joined by
     // the decay's powers (three launches); seg_state: float [entries, max_seg, heads, d, dv].
     if (entries <= 0) return 0;
@@ -433,7 +554,7 @@ extern "C" int se_retention_chunk(const float* q32, const float* k32, const void
         if (e != cudaSuccess) return (int)e;
         se::retention_chunk_kernel<T><<<grid, se::kChunkThreads, smem, stream>>>(
             q32, k32, (const T*)proj, proj_stride, v_off, decay, state, state_stride, cu_q, seq_rows, o, heads, d, dv,
-            max_seg, segments ? seg_len : 0, segments ? seg_state : nullptr);
+            max_seg, segments ? seg_len : 0, segments ? seg_state : nullptr, silu);
     });
     if (segments) {
         const int per = d * dv;
@@ -457,5 +578,23 @@ extern "C" int se_retention_out(const float* o, const void* proj, int proj_strid
     SE_DISPATCH_DTYPE(dtype, T,
         se::retention_out_kernel<T><<<(rows + 7) / 8, 256, 0, stream>>>(o, (const T*)proj, proj_stride, g_off, (T*)out,
                                                                          rows, heads, dv, eps));
+    SE_LAUNCH_CHECK();
+}
+
+// The joint form: one root mean square over the concatenated heads, a weight per column, a sigmoid gate.
+extern "C" int se_retention_out_joint(const float* o, const void* proj, int proj_stride, int g_off, const void* w, void* out,
+                                      int tokens, int width, float eps, int dtype, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (width <= 0) return SE_ERR_ARGUMENT;
+    const size_t esize = dtype == SE_DTYPE_F32 ? 4 : 2;
+    const int vec = width % 8 == 0 && (proj_stride * esize) % 16 == 0 && (g_off * esize) % 16 == 0 &&
+                    ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(w) |
+                      reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const int threads = width >= 4096 ? 256 : width >= 1024 ? 128 : 64;
+    SE_DISPATCH_DTYPE(dtype, T, {
+        cudaError_t e = SE_LAUNCH_DEPENDENT("ret", se::retention_out_joint_kernel<T>, dim3(tokens), dim3(threads), 0, stream, o,
+                                             (const T*)proj, proj_stride, g_off, (const T*)w, (T*)out, width, eps, vec);
+        if (e != cudaSuccess) return (int)e;
+    });
     SE_LAUNCH_CHECK();
 }

@@ -16,8 +16,8 @@ import torch
 from ..config.specs import ModelSpec, ParamSpec, Source
 from ..csrc import ops
 from ..parts.base import KVRequest, StateRequest, StepContext, make_norm
-from ..parts.block import (PostNormBlock, PreNormBlock, PreNormStreamBlock, StreamMixBlock, SublayerNormBlock,
-                           make_block)
+from ..parts.block import (PostNormBlock, PreNormBlock, PreNormStreamBlock, SandwichNormBlock, StreamMixBlock,
+                           SublayerNormBlock, make_block)
 from ..parts.linear import linear, linear32
 from ..parts.norm import RMSNorm
 
@@ -70,6 +70,12 @@ class Model:
                                         and hasattr(self.final_norm, "forward_stream")):
             raise ValueError("pre_norm_stream blocks need residual_stream='float32', a final norm with forward_stream, "
                              "and no other arrangement beside them")
+        # blocks with norms before and after each sublayer, which carry (result not yet normed and added, stream)
+        self.sandwich = any(isinstance(b, SandwichNormBlock) for b in self.blocks)
+        if self.sandwich and not (all(isinstance(b, SandwichNormBlock) for b in self.blocks) and spec.residual_stream == "float32"
+                                  and isinstance(self.final_norm, RMSNorm) and not self.final_norm.spec.offset):
+            raise ValueError("sandwich_norm blocks need residual_stream='float32', a plain RMS final norm, and no other "
+                             "arrangement beside them")
         # blocks over several 32-bit streams that carry (result not yet written, streams)
         self.multi_stream = any(isinstance(b, StreamMixBlock) for b in self.blocks)
         if self.multi_stream and not (all(isinstance(b, StreamMixBlock) for b in self.blocks)
@@ -188,7 +194,7 @@ class Model:
             e1.record()
             self.profile.setdefault(name, []).append((e0, e1))
             return out
-        if isinstance(block, StreamMixBlock):
+        if isinstance(block, (StreamMixBlock, SandwichNormBlock)):
             return block.forward(hidden, residual, step, slot, timed=timed)
         if isinstance(block, PreNormStreamBlock):
             return block.forward(hidden, residual, step, slot, inject=inject, timed=timed)
@@ -228,7 +234,7 @@ class Model:
             residual = torch.empty(step.num_tokens, s.streams, s.hidden_size, dtype=torch.float32, device=hidden.device)
             ops.stream_embed(self.embed, step.token_ids, residual, scale=s.embed_scale)
             hidden = None
-        elif pending_stream:
+        elif pending_stream or self.sandwich:
             # (output not yet added with its factor, 32-bit stream); `hidden` keeps the embedding output for the re-injections
             residual = torch.empty(hidden.shape, dtype=torch.float32, device=hidden.device)
             ops.embed_stream(self.embed, step.token_ids, residual,
@@ -274,6 +280,8 @@ class Model:
                 ops.stream_mix(both, write=hidden[0].write_args(hidden[1], hidden[2]), dtype=self.dtype)
                 self.stream_taps.append(ops.stream_sum(both, torch.empty(both.shape[0], both.shape[2], dtype=torch.float32,
                                                                          device=both.device)))
+            elif self.stream_taps is not None and self.sandwich:
+                self.stream_taps.append(SandwichNormBlock.settle(residual.clone(), hidden))
             elif self.stream_taps is not None:
                 tap = (residual if stream32 else hidden).float().clone()
                 if pending_stream and hidden is not None:
@@ -296,6 +304,8 @@ class Model:
             h = torch.empty(n, s.hidden_size, dtype=self.dtype, device=r.device)
             ops.stream_mix(r.view(n, s.streams, s.hidden_size), write=mix.write_args(yr, gr),
                            read=(None, self.final_norm.weight, self.final_norm.spec.eps, h), dtype=self.dtype, store=False)
+        elif self.sandwich:   # the last norm reads the wanted rows of the stream and of what it has not taken in yet
+            h = SandwichNormBlock.read(residual, hidden, self.final_norm, self.dtype, rows=want_rows)
         elif pending_stream:  # the wanted rows of the stream and of what it has not taken in yet
             r = torch.empty(n, s.hidden_size, dtype=torch.float32, device=residual.device)
             ops.gather_rows(residual, want_rows, r)

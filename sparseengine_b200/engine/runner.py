@@ -181,7 +181,7 @@ class ModelRunner:
             if end > self.cache.max_seq_len:
                 raise AssertionError(f"request {e.seq_id!r} would exceed the maximum length")
             for g in self.cache.groups:
-                lo = 0 if g.window is None else max(0, start - g.window + 1)
+                lo = g.request.first_visible(start)
                 idx = np.arange(lo // g.page_size, -(-end // g.page_size))
                 pages = g.table_host[row, idx]
                 if (pages < 0).any() or (pages >= g.pool.num_pages).any():

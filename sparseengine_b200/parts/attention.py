@@ -7,8 +7,8 @@ written before attention reads the cache.
 
 The general preparation (``prep="general"``) adds, each by a field of the spec: values of a head
 size of their own, a query temperature, layers without keys of their own, a cap on the scores,
-a sink of score 0 or of a learned score per head in the softmax, an output gate, values blended with
-those of an earlier layer, norms per head (with or without a weight), biases on the projections, a
+a sink of score 0 or of a learned score per head in the softmax, an output gate (per element or one number
+per head), keys of the query's own chunk only, values blended with those of an earlier layer, norms per head (with or without a weight), biases on the projections, a
 distance bias on the scores, and first positions that stay visible beside a window.  The blended values are what is cached; the earlier layer's values of this step's tokens
 travel from layer to layer in the step's scratch (``StepContext.extras``), so nothing of them
 is kept between steps.
@@ -20,7 +20,7 @@ import torch
 from ..config.specs import ParamSpec
 from ..csrc import ops
 from .base import KVRequest, Mixer, make_position, register_mixer
-from .linear import linear
+from .linear import linear, pad_rows
 from .position import RotaryArgs, as_rotary_args
 
 
@@ -41,18 +41,18 @@ class PagedAttention(Mixer):
         # hand `forward` the product's columns as `proj`); the rotary preparation reads a matrix of its own
         self.input_projection = "qkv" if self.general else None
         if self.general:
-            # no rotation; any head sizes the plain kernels take
+            # any head sizes the plain kernels take
             if not (0 < s.head_dim <= ops.LIMITS["attention_max_head_dim"]
                     and 0 < s.value_dim <= ops.LIMITS["attention_max_head_dim"]):
                 raise ValueError(f"head sizes {s.head_dim} / {s.value_dim} are not supported (1 to "
                                  f"{ops.LIMITS['attention_max_head_dim']})")
-            if s.position is not None and getattr(s.position, "pairing", "split_half") != "split_half":
-                raise ValueError("the general preparation rotates split halves only")
+            if s.position is not None and getattr(s.position, "pairing", "split_half") not in ("split_half", "interleaved"):
+                raise ValueError("the general preparation rotates split halves or neighbours in place")
             if s.q_temperature is not None and not (len(s.q_temperature) == 2 and int(s.q_temperature[1]) > 0):
                 raise ValueError("q_temperature is (coef, every) with every > 0")
         elif (s.v_head_dim not in (None, s.head_dim) or s.q_temperature is not None or not s.own_kv
               or s.score_softcap is not None or s.sink is not None or s.output_gate or s.value_mix is not None
-              or s.bias or s.keep_first or s.distance_slopes is not None or s.qk_norm in ("per_head", "per_head_unit")):
+              or s.bias or s.output_bias or s.keep_first or s.distance_slopes is not None or s.qk_norm in ("per_head", "per_head_unit")):
             raise ValueError("v_head_dim, q_temperature, own_kv=False, score_softcap, sink, output_gate, value_mix, "
                              "bias, keep_first, distance_slopes and per-head norms need prep='general'")
         elif s.head_dim <= 0 or s.head_dim % 16 or s.head_dim > ops.LIMITS["attention_max_head_dim"]:
@@ -67,10 +67,14 @@ class PagedAttention(Mixer):
             raise ValueError(f"distance_slopes needs one slope per query head ({s.num_heads}), got {len(s.distance_slopes)}")
         if s.keep_first < 0 or (s.keep_first and s.window is None):
             raise ValueError("keep_first is a count of first positions that stay visible beside a window")
-        if s.bias and (s.output_gate or not s.own_kv):
-            raise ValueError("biases go with projections of q, k and v alone")
+        if s.output_gate not in (False, True, "element", "head"):
+            raise ValueError(f"output_gate {s.output_gate!r} is not known (False, 'element' or 'head')")
+        if s.bias and not s.own_kv:
+            raise ValueError("biases go with projections of q, k and v")
         if s.window is not None and s.window <= 0:
             raise ValueError("window must be positive (None: all keys)")
+        if s.chunk is not None and (s.chunk <= 0 or s.window is not None):
+            raise ValueError("chunk must be positive (None: all keys) and stands in the place of a window")
         if s.score_softcap is not None and not s.score_softcap > 0:
             raise ValueError("score_softcap must be positive (None: no cap)")
         if s.sink not in (None, "zero", "learned"):
@@ -92,9 +96,8 @@ class PagedAttention(Mixer):
         s = self.spec
         q, kv = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
         rows = q + (kv + s.num_kv_heads * s.value_dim if s.own_kv else 0)
-        if s.output_gate:
-            rows += s.num_heads * s.value_dim
-        out = {"qkv": ParamSpec((rows, s.hidden_size)), "o": ParamSpec((s.hidden_size, s.num_heads * s.value_dim))}
+        gated = rows + self.gate_columns
+        out = {"qkv": ParamSpec((gated, s.hidden_size)), "o": ParamSpec((s.hidden_size, s.num_heads * s.value_dim))}
         if s.value_mix is not None:
             out["v_mix"] = ParamSpec((), "float32", "unit")
         if s.qk_norm in ("whole_projection", "per_head"):
@@ -104,15 +107,26 @@ class PagedAttention(Mixer):
                 out["k_norm"] = ParamSpec((s.head_dim if per_head else kv,), "act", "norm")
         if s.bias:
             out["qkv_bias"] = ParamSpec((rows,), "float32", "bias")
+        if s.bias if s.output_bias is None else s.output_bias:
             out["o_bias"] = ParamSpec((s.hidden_size,), "float32", "bias")
         if s.sink == "learned":
             out["sink"] = ParamSpec((s.num_heads,), "float32", "bias")
         return out
 
+    @property
+    def gate_columns(self) -> int:
+        s = self.spec
+        return 0 if not s.output_gate else s.num_heads * (1 if s.output_gate == "head" else s.value_dim)
+
+    def bind(self, tensors):
+        super().bind(tensors)
+        if self.general:
+            self.qkv = pad_rows(self.qkv)
+
     def kv_request(self):
         s = self.spec
         return KVRequest(s.num_kv_heads, s.head_dim, s.window, None if s.value_dim == s.head_dim else s.value_dim,
-                         keep_first=int(s.keep_first) if s.window is not None else 0)
+                         keep_first=int(s.keep_first) if s.window is not None else 0, chunk=s.chunk)
 
     def output_bias(self):
         """The output projection's bias (32-bit), for a caller that has set ``defer_output_bias``."""
@@ -130,12 +144,7 @@ class PagedAttention(Mixer):
             proj = linear(x, self.qkv)
         q_cols, kv_cols = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
         v_cols = s.num_kv_heads * s.value_dim
-        inv_freq, rotary_dim = None, 0
-        if self.position is not None:
-            rope = as_rotary_args(self.position.kernel_args(x.device))
-            if rope.scale != 1.0 or rope.pairing != "split_half":
-                raise ValueError("the general preparation rotates split halves without a factor on cos and sin")
-            inv_freq, rotary_dim = rope.inv_freq, rope.rotary_dim
+        rope = as_rotary_args(self.position.kernel_args(x.device)) if self.position is not None else RotaryArgs(None, 0)
         v_first = None
         if s.value_mix is not None:
             kept = step.extras.get(self.VALUE_MIX_KEY)
@@ -149,14 +158,15 @@ class PagedAttention(Mixer):
         ops.qk_prep_general(proj, self.q_norm, self.k_norm if s.own_kv else None, step.positions, step.token_seq,
                             step.seq_rows, slot.table, slot.kv, q, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads,
                             head_dim=s.head_dim, v_head_dim=s.value_dim, eps=s.qk_norm_eps, page_size=slot.page_size,
-                            has_kv=writes, temperature=s.q_temperature, inv_freq=inv_freq, rotary_dim=rotary_dim,
+                            has_kv=writes, temperature=s.q_temperature, inv_freq=rope.inv_freq, rotary_dim=rope.rotary_dim,
+                            pairing=rope.pairing, rope_scale=rope.scale,
                             v_first=v_first, v_mix=self.v_mix if v_first is not None else None, bias=self.qkv_bias,
                             per_head=s.qk_norm == "per_head", per_head_unit=s.qk_norm == "per_head_unit")
         attn = torch.empty(tokens, s.num_heads * s.value_dim, dtype=x.dtype, device=x.device)
         gate = None
         if s.output_gate:
             g0 = q_cols + (kv_cols + v_cols if s.own_kv else 0)
-            gate = proj[:, g0:g0 + s.num_heads * s.value_dim]
+            gate = proj[:, g0:g0 + self.gate_columns]
         # the kernel before the attention is the one that wrote q and this step's keys; it waited for the
         # projection (whose columns the gate is), and the step's inputs are older than both
         self.attend(q, attn, step, slot, after_qk_prep=True, gate=gate)
@@ -221,13 +231,14 @@ class PagedAttention(Mixer):
         ``gate``: the output gate's projection (a view with a row pitch), or None."""
         s = self.spec
         sink = self.sink if s.sink == "learned" else s.sink == "zero"
-        options = dict(v_head_dim=s.value_dim, softcap=s.score_softcap, sink=sink, gate=gate, keep_first=s.keep_first,
+        options = dict(v_head_dim=s.value_dim, softcap=s.score_softcap, sink=sink, gate=gate, keep_first=s.keep_first, chunk=s.chunk,
                        slopes=self.slopes(q.device))
         if (self.use_tensor_cores is not False and q.dtype == torch.bfloat16
                 and ops.attn_decode_supported(s.head_dim, s.num_heads, s.num_kv_heads)
                 and ops.attn_decode_value_dim_supported(s.value_dim)):
             if not self.takes_portion_kernel(step):
-                max_keys = step.max_kv_len if s.window is None else min(step.max_kv_len, s.window + s.keep_first)
+                most = s.chunk if s.chunk is not None else s.window + s.keep_first if s.window is not None else step.max_kv_len
+                max_keys = min(step.max_kv_len, most)
                 ops.attn_decode(q, slot.kv, slot.table, step.seq_rows, step.token_seq, step.positions, out,
                                 num_heads=s.num_heads, num_kv_heads=s.num_kv_heads, head_dim=s.head_dim,
                                 page_size=slot.page_size, scale=s.scale, window=s.window, max_keys=max_keys,

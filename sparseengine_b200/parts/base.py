@@ -13,8 +13,8 @@ the framework: call :func:`register_mixer` (or its siblings) before the model is
 
 What a mixer may ask of the cache manager:
 
-* :meth:`Mixer.kv_request` → :class:`KVRequest`: paged keys and values, all keys or a
-  window of them; layers whose requests are equal share one group of pages;
+* :meth:`Mixer.kv_request` → :class:`KVRequest`: paged keys and values, all keys, a
+  window or a chunk of them; layers whose requests are equal share one group of pages;
 * :meth:`Mixer.state_request` → :class:`StateRequest`: a per-request state of fixed
   size, zeroed when a request is admitted.
 """
@@ -39,6 +39,20 @@ class KVRequest:
     layout: str = "kv"
     # with a window: the first keep_first positions stay visible (and held) beside the window's
     keep_first: int = 0
+    # instead of a window: a query sees (and the cache keeps) only the positions of its own chunk of this many,
+    # counted from position 0
+    chunk: Optional[int] = None
+
+    @property
+    def bounded(self) -> bool:
+        """Whether old positions go out of sight."""
+        return self.window is not None or self.chunk is not None
+
+    def first_visible(self, position: int) -> int:
+        """The oldest position (beside kept first ones) that a query at ``position`` sees; it never falls."""
+        if self.window is not None:
+            return max(0, position - self.window + 1)
+        return position - position % self.chunk if self.chunk is not None else 0
 
     @property
     def value_dim(self) -> int:

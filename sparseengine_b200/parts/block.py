@@ -12,7 +12,8 @@ from ``LayerSpec.extra``.
 
 ``post_norm`` (:class:`PostNormBlock`), ``pre_norm_stream`` (:class:`PreNormStreamBlock`) and
 ``sublayer_norm`` (:class:`SublayerNormBlock`) are the arrangements over a 32-bit stream,
-``stream_mix`` (:class:`StreamMixBlock`) the one over several such streams.
+``stream_mix`` (:class:`StreamMixBlock`) the one over several such streams; ``sandwich_norm``
+(:class:`SandwichNormBlock`) norms before and after each sublayer.
 """
 from __future__ import annotations
 
@@ -218,7 +219,69 @@ class StreamMixBlock:
         return pending, streams
 
 
-ARRANGEMENTS = {"stream_mix": StreamMixBlock, "pre_norm": PreNormBlock, "post_norm": PostNormBlock, "pre_norm_stream": PreNormStreamBlock,
+class SandwichNormBlock:
+    """Norms before and after each sublayer, over a 32-bit stream: ``x <- x + post(mixer(norm(x)))``, then (if the
+    layer has a feed-forward) ``x <- x + post(feed_forward(norm(x)))``.  The block carries ``(pending, stream)``:
+    ``pending = (y, post norm)`` is the last sublayer's result that the stream has not taken in yet (None at the
+    start); the next sublayer's read norms it, adds it and norms the sum in one kernel (``ops.sandwich_norm``).  A mixer of
+    two normed branches leaves their sum to that kernel as well.  Whoever needs the stream itself (the
+    model's last norm, a tap) applies ``pending`` first (:meth:`read`)."""
+
+    def __init__(self, spec, dtype):
+        self.spec = spec
+        self.dtype = dtype
+        self.mixer = make_mixer(spec.mixer, dtype)
+        if hasattr(self.mixer, "defer_sum"):
+            self.mixer.defer_sum = True
+        self.feed_forward = make_feed_forward(spec.feed_forward, dtype) if spec.feed_forward is not None else None
+        norms = {"mixer_norm": spec.mixer_norm, "mixer_post_norm": spec.extra.get("mixer_post_norm")}
+        if self.feed_forward is not None:
+            norms.update({"feed_forward_norm": spec.feed_forward_norm,
+                          "feed_forward_post_norm": spec.extra.get("feed_forward_post_norm")})
+        self.norms = {}
+        for name, s in norms.items():
+            if getattr(s, "kind", None) != "rms" or s.offset or s.groups != 1:
+                raise ValueError(f"a sandwich_norm block needs a plain RMS norm as {name!r}")
+            self.norms[name] = make_norm(s, dtype)
+
+    def parts(self) -> dict:
+        out = {"mixer": self.mixer, **self.norms}
+        if self.feed_forward is not None:
+            out["feed_forward"] = self.feed_forward
+        return out
+
+    @staticmethod
+    def read(stream, pending, norm, dtype, rows=None, store=True):
+        """Apply ``pending`` to the stream (in place unless ``rows`` are asked for) and return its norm in the
+        activation type."""
+        from ..csrc import ops
+        y, post = pending if pending is not None else (None, None)
+        out = torch.empty(stream.shape[0] if rows is None else rows.numel(), stream.shape[1], dtype=dtype, device=stream.device)
+        return ops.sandwich_norm(stream, y, post=(post.weight, post.spec.eps) if post is not None else None,
+                                 following=(norm.weight, norm.spec.eps), out=out, rows=rows,
+                                 store=store and y is not None and rows is None)
+
+    @staticmethod
+    def settle(stream, pending):
+        """The stream with ``pending`` taken in."""
+        from ..csrc import ops
+        if pending is not None:
+            y, post = pending
+            ops.sandwich_norm(stream, y, post=(post.weight, post.spec.eps), dtype=(y[0][0] if isinstance(y, tuple) else y).dtype)
+        return stream
+
+    def forward(self, pending, stream, step, slot, timed=None):
+        run = timed if timed is not None else (lambda name, fn, *a: fn(*a))
+        h = run("mixer_norm", self.read, stream, pending, self.norms["mixer_norm"], self.dtype)
+        pending = (run("mixer." + self.mixer.spec.kind, self.mixer.forward, h, step, slot), self.norms["mixer_post_norm"])
+        if self.feed_forward is not None:
+            h = run("feed_forward_norm", self.read, stream, pending, self.norms["feed_forward_norm"], self.dtype)
+            pending = (run("feed_forward." + self.feed_forward.spec.kind, self.feed_forward.forward, h, step),
+                       self.norms["feed_forward_post_norm"])
+        return pending, stream
+
+
+ARRANGEMENTS = {"sandwich_norm": SandwichNormBlock, "stream_mix": StreamMixBlock, "pre_norm": PreNormBlock, "post_norm": PostNormBlock, "pre_norm_stream": PreNormStreamBlock,
                 "sublayer_norm": SublayerNormBlock}
 
 

@@ -49,6 +49,13 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, ac
     return y if activation is None else ops.activation_(y, activation)
 
 
+def pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """``w`` with zero rows added up to a multiple of ``multiple``: the product's rows then keep 16-byte alignment, also
+    where it is stacked with another matrix.  The added columns of the product are nobody's."""
+    extra = -w.shape[0] % multiple
+    return torch.cat([w, w.new_zeros(extra, *w.shape[1:])], 0) if extra else w
+
+
 def linear32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """x [rows, in] . w [out, in]^T with the result left in 32-bit (not rounded to the activation type):
     a product whose output joins a 32-bit residual stream."""

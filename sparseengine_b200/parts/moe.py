@@ -36,6 +36,8 @@ class _RoutedSwiGLU(FeedForward):
             raise ValueError(f"activation {spec.activation!r} is not supported; known: {sorted(ops.GLU_KINDS)}")
         if spec.activation == "silu":
             return None
+        if spec.activation == "gelu_tanh":
+            return (spec.activation, 0.0, 0.0)
         if not spec.activation_limit > 0:
             raise ValueError(f"activation {spec.activation!r} needs a positive activation_limit")
         return (spec.activation, float(spec.activation_limit), float(spec.activation_alpha))

@@ -1,5 +1,6 @@
 """Mixers side by side: every branch reads the same input, the result is the weighted sum of what
-they return (``config.specs.ParallelMixerSpec``).
+they return, or of that over its root mean square and times a weight (``output_norms``;
+``config.specs.ParallelMixerSpec``).
 
 A branch is any registered mixer.  The cache manager sees one mixer: the pages are the branch's that
 asks for pages, the state slot the branch's that asks for one (at most one each).  A branch that
@@ -8,11 +9,15 @@ has a bias on its output projection leaves it to the sum (one kernel: csrc/strea
 projects their input (``input_projection``) get one product for all of them: their matrices are
 stacked (the branches' own parameters become views of the stack) and each branch is handed its
 columns of the result.
+
+With ``output_norms`` the sum itself may be left to the block (``defer_sum``): ``forward`` then returns the
+branches' results with their weights and factors, the form that ``ops.sandwich_norm`` takes as one result.
 """
 from __future__ import annotations
 
 import torch
 
+from ..config.specs import ParamSpec
 from ..csrc import ops
 from .base import Mixer, make_mixer, register_mixer
 from .linear import linear
@@ -34,15 +39,23 @@ class ParallelMixer(Mixer):
         for b in self.branches:
             if hasattr(b, "defer_output_bias"):
                 b.defer_output_bias = True
+        if spec.output_norms and any(getattr(b.spec, "output_bias", None) or (getattr(b.spec, "bias", False) and getattr(b.spec, "output_bias", None) is None)
+                                     for b in self.branches):
+            raise ValueError("branches whose results are normed have no bias on their output projections")
+        self.defer_sum = False       # True: forward returns the branches' results for ops.sandwich_norm to add
         self._bias = None
         self._stacked = None         # the branches' input projections as one matrix, and where each one's rows start
 
     def parameters(self):
-        return {f"{name}_{k}": p for name, b in zip(self.spec.names, self.branches) for k, p in b.parameters().items()}
+        out = {f"{name}_{k}": p for name, b in zip(self.spec.names, self.branches) for k, p in b.parameters().items()}
+        if self.spec.output_norms:
+            out.update({f"{name}_out_norm": ParamSpec((self.spec.hidden_size,), "act", "norm") for name in self.spec.names})
+        return out
 
     def bind(self, tensors):
         for name, b in zip(self.spec.names, self.branches):
-            b.bind({k[len(name) + 1:]: v for k, v in tensors.items() if k.startswith(name + "_")})
+            b.bind({k[len(name) + 1:]: v for k, v in tensors.items() if k.startswith(name + "_") and k != name + "_out_norm"})
+        self._norms = [tensors[name + "_out_norm"] for name in self.spec.names] if self.spec.output_norms else None
         # the branches' output biases, weighed like the branches
         self._bias = None
         for a, b in zip(self.scales, self.branches):
@@ -77,6 +90,9 @@ class ParallelMixer(Mixer):
         else:
             y0 = self.branches[0].forward(x, step, slot)
             y1 = self.branches[1].forward(x, step, slot)
+        if self._norms is not None:
+            both = tuple((y, w, a) for y, w, a in zip((y0, y1), self._norms, self.scales)) + (self.spec.norm_eps,)
+            return both if self.defer_sum else ops.sandwich_norm(None, both, out=torch.empty_like(y0))
         return ops.scaled_sum(y0, y1, self.scales[0], self.scales[1], torch.empty_like(y0), bias=self._bias)
 
 

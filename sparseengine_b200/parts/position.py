@@ -109,9 +109,7 @@ def scaled_frequencies(rotary_dim: int, theta: float, scaling: Optional[dict]) -
     if bool(scaling.get("truncate", True)):
         first, last = math.floor(first), math.ceil(last)
     first, last = max(first, 0), min(last, rotary_dim - 1)
-    if first == last:
-        last += 0.001
-    ramp = torch.clamp((torch.arange(rotary_dim // 2, dtype=torch.float32) - first) / (last - first), 0, 1)
+    ramp = torch.clamp((torch.arange(rotary_dim // 2, dtype=torch.float32) - first) / max(last - first, 0.001), 0, 1)
     kept = 1 - ramp
     inv = inv / factor * (1 - kept) + inv * kept
     amplitude = scaling.get("attention_factor")

@@ -15,7 +15,7 @@ import torch
 from ..config.specs import ParamSpec
 from ..csrc import ops
 from .base import Mixer, StateRequest, make_position, register_mixer
-from .linear import linear
+from .linear import linear, pad_rows
 from .position import as_rotary_args
 
 
@@ -166,10 +166,14 @@ class GatedDeltaMixer(Mixer):
 
 
 class RetentionMixer(Mixer):
-    """``[q | k | v | g] = in_proj(h)``; q and k rotated by position, k times ``head_dim ** -0.5``; per
+    """``[q | k | v | g] = in_proj(h)``; q and k rotated by position, k times a factor; per
     head ``S <- decay S + k v^T``, ``o = S^T q`` with a fixed decay; each head's ``o`` over its root
     mean square, times ``silu(g)``; out projection (kernels: csrc/retention.cu).  The state is one
-    32-bit ``[heads, head_dim, v_head_dim]`` row per request."""
+    32-bit ``[heads, head_dim, v_head_dim]`` row per request.  Options (``config.specs.RetentionSpec``): q, k and v through
+    a silu first; one norm with a weight over the concatenated heads and a sigmoid gate."""
+    # the parameter that projects the mixer's input (a mixer of mixers may stack it with its neighbours' and
+    # hand `forward` the product's columns as `proj`)
+    input_projection = "in_proj"
     graph_safe = True
     chunk_min_tokens = 16        # the longest entry of a step from which the chunked kernel runs; None: never
 
@@ -185,6 +189,9 @@ class RetentionMixer(Mixer):
                              "a state column's rows live in the registers of eight warps)")
         if s.num_heads > ops.LIMITS["grid_dim_yz"]:
             raise ValueError("heads are a grid dimension of the kernels (at most 65,535)")
+        if s.activation not in (None, "silu") or s.output_norm not in ("per_head", "joint"):
+            raise ValueError("a retention mixer's activation is None or 'silu', its output_norm 'per_head' or 'joint'")
+        self.k_scale = float(s.k_scale) if s.k_scale is not None else s.head_dim ** -0.5
         self.position = make_position(s.position, dtype) if s.position is not None else None
         if self.position is not None:
             if s.position.pairing != "split_half":
@@ -197,14 +204,21 @@ class RetentionMixer(Mixer):
 
     def parameters(self):
         s = self.spec
-        return {"in_proj": ParamSpec((2 * self.qk + 2 * self.vv, s.hidden_size)),
-                "o": ParamSpec((s.hidden_size, self.vv))}
+        out = {"in_proj": ParamSpec((2 * self.qk + 2 * self.vv, s.hidden_size)),
+               "o": ParamSpec((s.hidden_size, self.vv))}
+        if s.output_norm == "joint":
+            out["norm_w"] = ParamSpec((self.vv,), "act", "norm")
+        return out
+
+    def bind(self, tensors):
+        super().bind(tensors)
+        self.in_proj = pad_rows(self.in_proj)
 
     def state_request(self):
         s = self.spec
         return StateRequest((s.num_heads * s.head_dim * s.v_head_dim,), torch.float32)
 
-    def forward(self, x, step, slot):
+    def forward(self, x, step, slot, proj=None):
         s = self.spec
         tokens, dev = x.shape[0], x.device
         if self._decay is None or self._decay.device != dev:
@@ -215,19 +229,27 @@ class RetentionMixer(Mixer):
             if rope.scale != 1.0:
                 raise ValueError("the retention kernels take no factor on cos and sin")
             inv_freq, rotary_dim = rope.inv_freq, rope.rotary_dim
-        proj = linear(x, self.in_proj)
-        q32 = torch.empty(tokens, self.qk, dtype=torch.float32, device=dev)
-        k32 = torch.empty(tokens, self.qk, dtype=torch.float32, device=dev)
-        ops.retention_prep(proj, 0, self.qk, inv_freq, step.positions, q32, k32, heads=s.num_heads, head_dim=s.head_dim,
-                           rotary_dim=rotary_dim, k_scale=s.head_dim ** -0.5)
+        if proj is None:
+            proj = linear(x, self.in_proj)
+        silu = s.activation == "silu"
         o = torch.empty(tokens, self.vv, dtype=torch.float32, device=dev)
         # a step with a prompt portion takes the recurrence in chunks of 64 tokens (closed form per chunk);
         # steps of single tokens and of short pieces walk it token by token
         chunked = self.chunk_min_tokens is not None and step.max_q_len >= self.chunk_min_tokens
-        (ops.retention_chunk if chunked else ops.retention_scan)(
-            q32, k32, proj, 2 * self.qk, self._decay, slot.state, step, o, heads=s.num_heads, head_dim=s.head_dim,
-            v_head_dim=s.v_head_dim)
+        args = (proj, 2 * self.qk, self._decay, slot.state, step, o)
+        sizes = dict(heads=s.num_heads, head_dim=s.head_dim, v_head_dim=s.v_head_dim, silu=silu)
+        if not chunked and rotary_dim == 0:      # q and k straight from the projection, as they are staged
+            ops.retention_scan(None, None, *args, **sizes, qk=(0, self.qk, self.k_scale))
+        else:
+            q32 = torch.empty(tokens, self.qk, dtype=torch.float32, device=dev)
+            k32 = torch.empty(tokens, self.qk, dtype=torch.float32, device=dev)
+            ops.retention_prep(proj, 0, self.qk, inv_freq, step.positions, q32, k32, heads=s.num_heads, head_dim=s.head_dim,
+                               rotary_dim=rotary_dim, k_scale=self.k_scale, silu=silu)
+            (ops.retention_chunk if chunked else ops.retention_scan)(q32, k32, *args, **sizes)
         gated = torch.empty(tokens, self.vv, dtype=x.dtype, device=dev)
+        if s.output_norm == "joint":
+            ops.retention_out_joint(o, proj, 2 * self.qk + self.vv, self.norm_w, gated, eps=s.norm_eps)
+            return linear(gated, self.o)
         ops.retention_out(o, proj, 2 * self.qk + self.vv, gated, heads=s.num_heads, v_head_dim=s.v_head_dim, eps=s.norm_eps)
         return linear(gated, self.o)
 
