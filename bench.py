@@ -482,7 +482,7 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-long-context", action="store_true", help="leave out the 131,072-token point")
     ap.add_argument("--long-layers", type=int, default=LONG_LAYERS)
-    ap.add_argument("--design", default="minimax_m2", choices=["minimax_m2", "hybrid", "zisevik", "kisusun", "tedisun", "nurolorn"],
+    ap.add_argument("--design", default="minimax_m2", choices=["minimax_m2", "hybrid", "zisevik", "kisusun", "tedisun", "nurolorn", "movivik"],
                     help="hybrid: prefill and decode throughput of the hybrid design (attention, state-space and "
                          "gated-delta mixers) at two layer sizes beside MiniMax M2 layers of equal width, and its "
                          "kernels alone against their rooflines, instead of the headline workload; zisevik: the same "
@@ -492,7 +492,9 @@ def main() -> int:
                          "(several residual streams, a delta rule with one decay per head, attention with kept first keys and "
                          "a learned sink beside a matrix memory, identity experts) beside the Zisevik design; nurolorn: the "
                          "same for the Nurolorn design (latent attention with a gate, minGRU, windowed attention with a "
-                         "distance bias, a looped stack) beside the Zisevik design with dense feed-forwards")
+                         "distance bias, a looped stack) beside the Zisevik design with dense feed-forwards; movivik: the "
+                         "same for the Movivik design (attention within chunks, full attention beside lightning "
+                         "attention, norms around each sublayer) beside the Tedisun design")
     ap.add_argument("--only-decode", action="store_true",
                     help="time the headline decode only (no points, prefill or end-to-end run): for profiling")
     args = ap.parse_args()
@@ -528,6 +530,10 @@ def main() -> int:
     if args.design == "nurolorn":
         from sparseengine_b200.cli import nurolorn_bench
         print(json.dumps(nurolorn_bench.run(steps=min(args.steps, 20), warmup=args.warmup)))
+        return 0
+    if args.design == "movivik":
+        from sparseengine_b200.cli import movivik_bench
+        print(json.dumps(movivik_bench.run(steps=min(args.steps, 20), warmup=args.warmup)))
         return 0
     if args.design == "kisusun":
         from sparseengine_b200.cli import kisusun_bench

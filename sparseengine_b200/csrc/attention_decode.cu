@@ -12,7 +12,7 @@
 // 32-bit, probabilities rounded to bfloat16 before they multiply V, the output rounded once.
 //
 // Any page size; query/key and value head sizes that are multiples of 8 up to 128 (others use the plain
-// kernel): tiles have 64 or 128 query/key columns and 32, 64 or 128 value columns, and a head size between
+// kernel), from 40 and 24 on (a narrower head would leave most of its tile empty): tiles have 64 or 128 query/key columns and 32, 64 or 128 value columns, and a head size between
 // them lies in the next wider tile, the columns beyond it zero.  A window (with or without first keys that
 // stay visible) or a chunk (first_visible) is honoured.  A page holds the keys [kv head][slot][D] and then the values
 // [kv head][slot][DV].  The softmax's options (a cap on the scores, a sink, an output gate, a distance bias)
@@ -337,11 +337,11 @@ static int launch(const void* q, const void* cache, const int* table, int table_
 }  // namespace se
 
 extern "C" int se_attn_decode_supported(int head_dim, int hq, int hkv) {
-    return (head_dim > 0 && head_dim <= 128 && head_dim % 8 == 0 && hkv > 0 && hq % hkv == 0) ? 1 : 0;
+    return (head_dim > 32 && head_dim <= 128 && head_dim % 8 == 0 && hkv > 0 && hq % hkv == 0) ? 1 : 0;
 }
 // the value head sizes the kernel takes beside a query/key head size it takes
 extern "C" int se_attn_decode_value_dim_supported(int v_head_dim) {
-    return (v_head_dim > 0 && v_head_dim <= 128 && v_head_dim % 8 == 0) ? 1 : 0;
+    return (v_head_dim > 16 && v_head_dim <= 128 && v_head_dim % 8 == 0) ? 1 : 0;
 }
 
 // part_o: float [tokens, hq, splits, v_head_dim]; part_ml: float [tokens, hq, splits, 2] (unused when splits == 1).

@@ -12,7 +12,7 @@
 // src/sparseengine/kernels/triton/context_flashattention_nopad.py:92-127.
 //
 // Any page size; query/key and value head sizes that are multiples of 8 up to 128 (others use the plain
-// kernel): tiles have 64 or 128 query/key columns and 32, 64 or 128 value columns, and a head size between
+// kernel), from 40 and 24 on (a narrower head would leave most of its tile empty): tiles have 64 or 128 query/key columns and 32, 64 or 128 value columns, and a head size between
 // them lies in the next wider tile, the columns beyond it zero.  Instead of a window, a chunk may bound
 // the keys (first_visible).  A page holds the keys [kv head][slot][D] and then the values [kv head][slot][DV].
 // The softmax's options (a cap on the scores, a sink, an output gate, a distance bias) are those of
@@ -328,7 +328,7 @@ extern "C" int se_attn_prefill(const void* q, const void* cache, const int* tabl
                                int gate_pitch, const float* sink_logits, int keep_first, const float* slopes,
                                int gate_per_head, cudaStream_t stream) {
     if (entries <= 0 || max_q_len <= 0) return 0;
-    if (head_dim <= 0 || head_dim > 128 || head_dim % 8 || v_head_dim <= 0 || v_head_dim > 128 || v_head_dim % 8 || hkv <= 0 || hq % hkv || entries > 65535 || hkv > 65535)
+    if (head_dim <= 32 || head_dim > 128 || head_dim % 8 || v_head_dim <= 16 || v_head_dim > 128 || v_head_dim % 8 || hkv <= 0 || hq % hkv || entries > 65535 || hkv > 65535)
         return SE_ERR_UNSUPPORTED;
     if (softcap < 0.f || !(scale > 0.f) || (gate != nullptr && gate_pitch < (gate_per_head ? hq : hq * v_head_dim)) || keep_first < 0)
         return SE_ERR_ARGUMENT;

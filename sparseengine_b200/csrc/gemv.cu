@@ -9,7 +9,11 @@
 // harmless because A and B use the same permutation and the sum over k does not care.  No
 // shared memory on the way in; the 8 or 16 warps of a block split K and add their partial
 // sums through shared memory at the end.  The weights are read exactly once.
+//
+// With GLU the fragment's lower 8 rows are rows of the gate matrix and its upper 8 the same rows of the up matrix (which
+// follows it in memory), so a block has both products of its outputs and applies the gated activation itself.
 #include "common.cuh"
+#include "glu.cuh"
 #include "mma_util.cuh"
 #include <cstdlib>
 
@@ -27,19 +31,21 @@ namespace gemv {
 #define SE_GEMV_PRELOAD 4
 #endif
 
-template <int NT, int kWarps, int kRowsPerBlock>
+template <int NT, int kWarps, int kRowsPerBlock, bool GLU = false>
 __global__ void __launch_bounds__(32 * kWarps)
 gemv_kernel(const __nv_bfloat16* x, const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
-            int rows, int n_out, int k_dim, int act) {
+            int rows, int n_out, int k_dim, int act, float limit, float alpha) {
     grid_dependency_trigger();       // the kernel after this one may set itself up meanwhile
     constexpr int kPreload = SE_GEMV_PRELOAD;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t4 = lane & 3;
-    const int n0 = blockIdx.x * kRowsPerBlock;
+    static_assert(!GLU || kRowsPerBlock == 16, "gate rows and up rows fill a fragment");
+    constexpr int kOutsPerBlock = GLU ? 8 : kRowsPerBlock;
+    const int n0 = blockIdx.x * kOutsPerBlock;
     const int chunks = k_dim / 32;
     const int c_begin = warp * chunks / kWarps, c_end = (warp + 1) * chunks / kWarps;
     const __nv_bfloat16* w_lo = w + (size_t)min(n0 + g, n_out - 1) * k_dim + 8 * t4;
-    const __nv_bfloat16* w_hi = w + (size_t)min(n0 + g + 8, n_out - 1) * k_dim + 8 * t4;
+    const __nv_bfloat16* w_hi = w + (size_t)(GLU ? n_out + min(n0 + g, n_out - 1) : min(n0 + g + 8, n_out - 1)) * k_dim + 8 * t4;
     const __nv_bfloat16* x_row[NT];
     bool x_ok[NT];
 #pragma unroll
@@ -97,12 +103,20 @@ gemv_kernel(const __nv_bfloat16* x, const __nv_bfloat16* __restrict__ w, __nv_bf
         }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < kRowsPerBlock * 8 * NT; i += blockDim.x) {
-        const int r = i % kRowsPerBlock, t = i / kRowsPerBlock;      // consecutive threads -> consecutive n
+    for (int i = threadIdx.x; i < kOutsPerBlock * 8 * NT; i += blockDim.x) {
+        const int r = i % kOutsPerBlock, t = i / kOutsPerBlock;      // consecutive threads -> consecutive n
         if (t < rows && n0 + r < n_out) {
             float v = 0.f;
 #pragma unroll
             for (int wq = 0; wq < kWarps; ++wq) v += part[wq][r][t];
+            if (GLU) {
+                float u = 0.f;
+#pragma unroll
+                for (int wq = 0; wq < kWarps; ++wq) u += part[wq][(r + 8) % kRowsPerBlock][t];
+                out[(size_t)t * n_out + n0 + r] = __float2bfloat16_rn(
+                    glu_value<__nv_bfloat16>(round_act<__nv_bfloat16>(v), round_act<__nv_bfloat16>(u), act, limit, alpha));
+                continue;
+            }
             const __nv_bfloat16 y = __float2bfloat16_rn(v);
             // as a product and an activation in two kernels would: the activation reads the rounded product
             out[(size_t)t * n_out + n0 + r] = act >= 0 ? __float2bfloat16_rn(act_apply(__bfloat162float(y), act)) : y;
@@ -120,7 +134,7 @@ extern "C" int se_gemv_supported(int rows, int n_out, int k_dim) {
 template <int NT, int W, int R>
 static void launch_gemv(const void* x, const void* w, void* out, int rows, int n_out, int k_dim, int act, cudaStream_t stream) {
     SE_LAUNCH_DEPENDENT("gemv", se::gemv::gemv_kernel<NT, W, R>, dim3(se::ceil_div(n_out, R)), dim3(32 * W), 0, stream,
-                         (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, rows, n_out, k_dim, act);
+                         (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, rows, n_out, k_dim, act, 0.f, 0.f);
 }
 
 // x [rows <= 16, k_dim], w [n_out, k_dim], out [rows, n_out]; bf16; k_dim a multiple of 32.  act: -1 none, else the
@@ -145,5 +159,21 @@ extern "C" int se_gemv(const void* x, const void* w, void* out, int rows, int n_
         default: return SE_ERR_ARGUMENT;
     }
 #undef SE_GEMV_CASE
+    SE_LAUNCH_CHECK();
+}
+
+// w [2 * n_out, k_dim]: gate rows, then up rows; out [rows, n_out] = the gated activation (glu.cuh) of the two rounded products.
+extern "C" int se_gemv_glu(const void* x, const void* w, void* out, int rows, int n_out, int k_dim, int kind, float limit, float alpha,
+                           cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (kind < SE_GLU_SILU || kind > SE_GLU_GELU) return SE_ERR_ARGUMENT;
+    if (!se_gemv_supported(rows, n_out, k_dim)) return SE_ERR_UNSUPPORTED;
+#define SE_GEMV_GLU(NT, W)                                                                                                  \
+    SE_LAUNCH_DEPENDENT("gemv", (se::gemv::gemv_kernel<NT, W, 16, true>), dim3(se::ceil_div(n_out, 8)), dim3(32 * W), 0, stream, \
+                         (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, rows, n_out, k_dim, kind, limit, alpha)
+    const cudaError_t e = rows <= 8 ? (k_dim >= 4096 ? SE_GEMV_GLU(1, 16) : SE_GEMV_GLU(1, 8))
+                                    : (k_dim >= 4096 ? SE_GEMV_GLU(2, 16) : SE_GEMV_GLU(2, 8));
+#undef SE_GEMV_GLU
+    if (e != cudaSuccess) return (int)e;
     SE_LAUNCH_CHECK();
 }

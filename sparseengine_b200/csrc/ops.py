@@ -1142,7 +1142,7 @@ def gemm_tc_dense(x, w, out, nt: int = 128):
 def attn_decode_supported(head_dim: int, num_heads: int, num_kv_heads: int) -> bool:
     """What ``se_attn_decode_supported`` of the library answers, restated here so that asking does not
     compile the kernel for a model that cannot use it (a GPU test compares the two)."""
-    return 0 < head_dim <= 128 and head_dim % 8 == 0 and num_kv_heads > 0 and num_heads % num_kv_heads == 0
+    return 32 < head_dim <= 128 and head_dim % 8 == 0 and num_kv_heads > 0 and num_heads % num_kv_heads == 0
 
 
 _sm_counts: dict = {}
@@ -1195,7 +1195,7 @@ def _softmax_options(q, gate, num_heads, v_head_dim, softcap, sink, keep_first, 
 
 def attn_decode_value_dim_supported(v_head_dim: int) -> bool:
     """Value head sizes the tensor-core kernels take beside a query/key head size they take."""
-    return 0 < v_head_dim <= 128 and v_head_dim % 8 == 0
+    return 16 < v_head_dim <= 128 and v_head_dim % 8 == 0
 
 
 def attn_decode(q, cache, table, seq_rows, token_seq, positions, out, *, num_heads, num_kv_heads, head_dim, page_size,
@@ -1274,6 +1274,28 @@ def gemv(x, w, out, activation=None):
     _check(_fn("se_gemv", "pppiiiip")(
         _ptr(x, torch.bfloat16, "x"), _ptr(w, torch.bfloat16, "w"), _ptr(out, torch.bfloat16, "out"), rows, n_out,
         k_dim, -1 if activation is None else ACTIVATIONS[activation], _stream()), "gemv")
+    return out
+
+
+def gemv_glu(x, w, out, activation=None):
+    """out[rows <= 16, n] = glu(x · w[:n]ᵀ, x · w[n:]ᵀ): gate rows, then up rows of one matrix, both products rounded before
+    the gated activation (``activation`` as :func:`glu`'s)."""
+    rows, k_dim = x.shape
+    n_out = w.shape[0] // 2
+    _check(_fn("se_gemv_glu", "pppiiiiffp")(
+        _ptr(x, torch.bfloat16, "x"), _ptr(w, torch.bfloat16, "w"), _ptr(out, torch.bfloat16, "out"), rows, n_out,
+        k_dim, *_glu_args(activation), _stream()), "gemv_glu")
+    return out
+
+
+def glu(x, out, activation=None):
+    """out[rows, n] = the gated activation of x[rows, 2n] = [gate | up] (32-bit arithmetic, rounded once; csrc/glu.cu).
+    ``activation``: a name of :data:`GLU_KINDS`, or ``(name, limit, alpha)``."""
+    rows, width = out.shape
+    if x.shape != (rows, 2 * width) or x.dtype != out.dtype:
+        raise ValueError("glu: x must be [rows, 2 * width] of out's type")
+    _check(_fn("se_glu", "ppiiiffip")(_ptr(x, None, "x"), _ptr(out, None, "out"), rows, width, *_glu_args(activation),
+                                      dtype_code(x.dtype), _stream()), "glu")
     return out
 
 

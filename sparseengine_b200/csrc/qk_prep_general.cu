@@ -248,17 +248,18 @@ __global__ void __launch_bounds__(kPrepItems)
 qk_prep_heads_kernel(const T* proj, int pitch, const T* __restrict__ q_w, const T* __restrict__ k_w,
                      const float* __restrict__ inv_freq, int rotary_dim, float rope_scale, const float* __restrict__ bias,
                      const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ seq_rows,
-                     const int* __restrict__ table, int table_stride, T* cache, T* q_out, long long items, int hq, int hkv,
+                     const int* __restrict__ table, int table_stride, T* cache, T* q_out, unsigned items, int hq, int hkv,
                      int d, int dv, float eps, int page_size, int num_pages, int* __restrict__ error) {
     extern __shared__ float2 turns[];            // [tokens of the block][rotary_dim / 2]: (cos, sin) * rope_scale
     grid_dependency_trigger();
     const int lanes = d / 8, qc = hq * lanes, kc = hkv * lanes, per_token = qc + kc + hkv * (dv / 8);
-    const long long x0 = (long long)blockIdx.x * kPrepItems, x = x0 + threadIdx.x;
+    const unsigned x0 = blockIdx.x * kPrepItems, x = x0 + threadIdx.x;
     const int t_first = (int)(x0 / per_token), half = rotary_dim / 2;
+    const int from = (int)(x0 - (unsigned)t_first * per_token);       // the block's first item within its first token
     grid_dependency_wait();
     if (ROT) {
-        const long long last = x0 + kPrepItems - 1 < items ? x0 + kPrepItems - 1 : items - 1;
-        const int n = ((int)(last / per_token) - t_first + 1) * half;
+        const int count = (int)min((unsigned)kPrepItems, items - x0);
+        const int n = ((from + count - 1) / per_token + 1) * half;
         for (int i = threadIdx.x; i < n; i += kPrepItems) {
             const int t = i / half;
             float sn, cs;
@@ -267,8 +268,9 @@ qk_prep_heads_kernel(const T* proj, int pitch, const T* __restrict__ q_w, const 
         }
     }
     const bool live = x < items;
-    const int t = live ? (int)(x / per_token) : t_first;
-    const int c = live ? (int)(x - (long long)t * per_token) : 0;
+    const int ahead = live ? (from + (int)threadIdx.x) / per_token : 0;
+    const int t = t_first + ahead;
+    const int c = live ? from + (int)threadIdx.x - ahead * per_token : 0;
     const T* row = proj + (size_t)t * pitch;
     auto load_raw = [&](int chunk, float* v) {
         load8(row + 8 * chunk, v);
@@ -374,14 +376,14 @@ extern "C" int se_qk_prep_general(const void* proj, int pitch, const void* q_w, 
         aligned(q_out) && aligned(cache) && aligned(q_w) && aligned(k_w) && aligned(bias)) {
         const long long items = (long long)tokens * per_token;
         const long long blocks = (items + se::kPrepItems - 1) / se::kPrepItems;
-        if (blocks > 0x7fffffffLL) return SE_ERR_UNSUPPORTED;
+        if (items > 0x7fffff00LL) return SE_ERR_UNSUPPORTED;
         const size_t turns = rotary_dim > 0 ? (size_t)se::prep_block_tokens(per_token) * (rotary_dim / 2) * sizeof(float2) : 0;
         const int norm = per_head, rot = rotary_dim == 0 ? 0 : interleaved ? 2 : 1;
 #define SE_PREP_CASE(N, R)                                                                                                  \
     if (norm == N && rot == R)                                                                                              \
         e = SE_LAUNCH_DEPENDENT("qk", (se::qk_prep_heads_kernel<T, N, R>), dim3((unsigned)blocks), dim3(se::kPrepItems), turns, stream, \
                                  (const T*)proj, pitch, (const T*)q_w, (const T*)k_w, inv_freq, rotary_dim, rope_scale, bias, \
-                                 positions, token_seq, seq_rows, table, table_stride, (T*)cache, (T*)q_out, items, hq, hkv, d, \
+                                 positions, token_seq, seq_rows, table, table_stride, (T*)cache, (T*)q_out, (unsigned)items, hq, hkv, d, \
                                  dv, eps, page_size, num_pages, error);
         SE_DISPATCH_DTYPE(dtype, T, {
             cudaError_t e = cudaErrorInvalidValue;

@@ -259,8 +259,8 @@ template <typename T, int NY>
 static cudaError_t launch(const Args& a, int rows, bool vec, cudaStream_t stream) {
     const int chunks = a.hidden / 8;
     if (vec && chunks <= 4 * kMaxThreads) {
-        // few rows: as many threads as there are chunks (a row's latency is what counts); many rows: two chunks a thread
-        const int want = rows >= 1024 && chunks >= 256 ? (chunks + 1) / 2 : chunks;
+        // few rows, and two results: as many threads as there are chunks; many rows of one result: two chunks a thread
+        const int want = NY < 2 && rows >= 1024 && chunks >= 256 ? (chunks + 1) / 2 : chunks;
         int threads = (want + 31) / 32 * 32;
         if (threads > kMaxThreads) threads = kMaxThreads;
         const int ch = (chunks + threads - 1) / threads;

@@ -29,6 +29,7 @@ GEMV_MAX_OUT = 16384
 # 16 rows 4,503 against 4,423: the kernel's second 8-row tile costs more than the library's
 # product, which for 17 to 128 rows takes 11 µs per projection).  ``gemv_max_rows`` sets it.
 GEMV_MAX_ROWS = 8
+GEMV_GLU_MAX_OUT = 65536       # gate and up rows together
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, activation: str | None = None) -> torch.Tensor:
@@ -47,6 +48,17 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, ac
         return ops.gemv(x, w, out, activation)
     y = torch.matmul(x, w.t()) if out is None else torch.matmul(x, w.t(), out=out)
     return y if activation is None else ops.activation_(y, activation)
+
+
+def linear_glu(x: torch.Tensor, w: torch.Tensor, activation=None) -> torch.Tensor:
+    """The gated activation of x [rows, in] . w [2n, in]^T (gate rows, then up rows) -> [rows, n]: inside this library's
+    few-row kernel, else as a kernel of its own after the library product.  ``activation`` as ``ops.glu``'s."""
+    n = w.shape[0] // 2
+    out = torch.empty(x.shape[0], n, dtype=x.dtype, device=x.device)
+    if (USE_GEMV and x.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and x.shape[0] <= GEMV_MAX_ROWS
+            and w.shape[0] <= GEMV_GLU_MAX_OUT and ops.gemv_supported(x.shape[0], n, x.shape[1])):
+        return ops.gemv_glu(x, w, out, activation)
+    return ops.glu(torch.matmul(x, w.t()), out, activation)
 
 
 def pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:

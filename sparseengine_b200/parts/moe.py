@@ -14,6 +14,7 @@ import torch
 from ..config.specs import ParamSpec
 from ..csrc import ops
 from .base import FeedForward, register_feed_forward
+from .linear import linear, linear_glu
 
 
 class _RoutedSwiGLU(FeedForward):
@@ -278,16 +279,20 @@ class SparseMoE(_RoutedSwiGLU):
                           for a in range(0, x.shape[0], self.chunk_rows)], 0)
 
 
-class DenseMLP(_RoutedSwiGLU):
-    """SwiGLU MLP = one expert every token selects with weight 1."""
+class DenseMLP(FeedForward):
+    """A dense gated feed-forward: one product for gate and up, the gated activation, one product down.
+
+    Measured at widths of 2,048 and 4,096 (feed-forward 4 x width; microseconds, 64 / 2,048 / 8,192 rows at 4,096): the
+    library products 78 / 531 / 2,299 and the activation beside them, the experts' kernels with one expert 216 / 669 /
+    3,084."""
+
+    graph_safe = True
 
     def __init__(self, spec, dtype):
         super().__init__(spec, dtype)
-        self.activation_args = self.activation_of(spec)
+        self.activation_args = _RoutedSwiGLU.activation_of(spec)
         if spec.hidden_size <= 0 or spec.intermediate_size <= 0:
             raise ValueError("hidden_size and intermediate_size must be positive")
-        self.num_experts, self.top_k = 1, 1
-        self.hidden, self.inter = spec.hidden_size, spec.intermediate_size
 
     def parameters(self):
         s = self.spec
@@ -295,10 +300,7 @@ class DenseMLP(_RoutedSwiGLU):
                 "w2": ParamSpec((1, s.hidden_size, s.intermediate_size))}
 
     def forward(self, x, step):
-        tokens = x.shape[0]
-        ids = torch.zeros(tokens, 1, dtype=torch.int32, device=x.device)
-        weights = torch.ones(tokens, 1, dtype=torch.float32, device=x.device)
-        return self.run_experts(x, ids, weights)
+        return linear(linear_glu(x, self.w13[0], self.activation_args), self.w2[0])
 
 
 register_feed_forward("moe", SparseMoE)
