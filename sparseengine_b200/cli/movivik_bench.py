@@ -204,7 +204,7 @@ def run(sizes=(2048, 4096), steps: int = 20, warmup: int = 3, kernels: bool = Tr
             one["movivik_parts_ms"] = _parts(mine, 2048, 8)
             one["closest_parts_ms"] = _parts(other, 2048, 8)
         if kernels:
-            one["kernels"] = _kernels(width, [(2048, 1, 0), (8192, 4, 0), (64, 64, 2048)], pk)
+            one["kernels"] = _kernels(width, [(2048, 1, 0), (8192, 4, 0), (64, 64, 3000)], pk)
         rec["sizes"][str(width)] = one
     return rec
 
