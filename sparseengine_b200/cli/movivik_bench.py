@@ -120,7 +120,7 @@ def _attention_kernels(width, tokens, entries, held, step, kv_len, add):
     hkv = max(1, hq // 4)
     pages = -(-(held + per) // PAGE_SIZE)
     table = torch.arange(entries * pages, device=dev, dtype=torch.int32).view(entries, pages)
-    for d, dv in ((128, 128), (96, 48)):
+    for d, dv in ((128, 128), (96, 64)):
         qn, kn, vn = hq * d, hkv * d, hkv * dv
         cache = (torch.randn(entries * pages, PAGE_SIZE * hkv * (d + dv), device=dev) * 0.5).to(bf)
         proj = torch.randn(tokens, qn + kn + vn + (hq + 7) // 8 * 8, device=dev, dtype=bf)

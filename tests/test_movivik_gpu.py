@@ -450,7 +450,7 @@ def held(cache, b, e, page, kv_heads, d, dv):
 
 
 @pytest.mark.parametrize("d,dv,heads,kv_heads,chunk,window,gated", [
-    (64, 64, 4, 2, 33, None, "head"), (128, 64, 6, 1, 70, None, "head"), (96, 48, 6, 2, 50, None, "head"), (40, 24, 3, 3, 17, None, "head"),
+    (64, 64, 4, 2, 33, None, "head"), (128, 64, 6, 1, 70, None, "head"), (104, 56, 6, 2, 50, None, "head"), (40, 24, 3, 3, 17, None, "head"),
     (128, 128, 8, 2, 100, None, "head"), (128, 128, 6, 6, 1, None, "head"), (128, 128, 4, 1, None, None, "head"), (72, 128, 20, 1, 64, None, None),
     (88, 104, 4, 2, None, 37, "element"), (120, 32, 2, 1, None, None, "element"), (128, 128, 4, 2, 64, None, "element"), (56, 40, 34, 2, 90, None, "head")])
 def test_chunks_gates_and_head_sizes_in_the_attention_kernels(d, dv, heads, kv_heads, chunk, window, gated):
@@ -503,13 +503,13 @@ def test_chunks_gates_and_head_sizes_in_the_attention_kernels(d, dv, heads, kv_h
 
 
 @pytest.mark.parametrize("d,dv,heads,kv_heads,rot,pairing,norm,bias,scale", [
-    (96, 48, 6, 2, 96, "interleaved", None, True, 1.3), (64, 64, 4, 1, 16, "split_half", "unit", False, 1.0),
+    (104, 56, 6, 2, 104, "interleaved", None, True, 1.3), (64, 64, 4, 1, 16, "split_half", "unit", False, 1.0),
     (128, 128, 8, 2, 64, "split_half", "unit", False, 1.4), (128, 40, 4, 4, 128, "interleaved", "unit", True, 0.7),
     (64, 24, 3, 1, 64, "split_half", "weights", True, 1.1), (256, 64, 4, 2, 32, "interleaved", "weights", False, 1.2),
     (16, 16, 2, 2, 16, "split_half", "unit", False, 1.5), (8, 8, 1, 1, 8, "interleaved", "unit", True, 1.5), (40, 16, 5, 1, 32, "split_half", None, True, 1.0),
     # sizes that leave the chunked kernel
-    (12, 20, 4, 2, 6, "split_half", "unit", False, 1.4), (10, 3, 5, 5, 6, "interleaved", None, True, 1.2), (96, 48, 6, 2, 32, "split_half", "unit", True, 1.6),
-    (96, 48, 3, 1, 24, "interleaved", "unit", False, 1.6), (13, 7, 3, 1, 4, "interleaved", "weights", True, 0.8), (24, 24, 2, 1, 0, "split_half", "unit", True, 1.0)])
+    (12, 20, 4, 2, 6, "split_half", "unit", False, 1.4), (10, 3, 5, 5, 6, "interleaved", None, True, 1.2), (104, 56, 6, 2, 32, "split_half", "unit", True, 1.6),
+    (104, 56, 3, 1, 24, "interleaved", "unit", False, 1.6), (13, 7, 3, 1, 4, "interleaved", "weights", True, 0.8), (24, 24, 2, 1, 0, "split_half", "unit", True, 1.0)])
 def test_query_and_key_preparation(d, dv, heads, kv_heads, rot, pairing, norm, bias, scale):
     """Biases, rotations of both pairings with a factor on cos and sin, and norms per head (over the rotated head
     where they have no weights) against the equations; queries, keys and values in their places."""
